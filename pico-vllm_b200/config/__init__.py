@@ -3,7 +3,10 @@ from .qwen2 import Qwen2Config
 from .zapipel import ZapipelConfig
 from .zikupel import ZikupelConfig
 from .zazilix import ZazilixConfig
+from .banazen import BanazenConfig
+from .vanapel import VanapelConfig
 from .engine import EngineConfig, canonical_dtype
 
-__all__ = ["KeyReader", "read_config_json", "architecture_name", "Qwen2Config", "ZapipelConfig", "ZikupelConfig", "ZazilixConfig", "EngineConfig",
+__all__ = ["KeyReader", "read_config_json", "architecture_name", "Qwen2Config", "ZapipelConfig", "ZikupelConfig", "ZazilixConfig", "BanazenConfig",
+           "VanapelConfig", "EngineConfig",
            "canonical_dtype"]

@@ -1,5 +1,5 @@
 // Paged causal attention with grouped heads, for any head size that is a multiple of 16 up to
-// 256, float32 or bfloat16 storage, float32 arithmetic.  One block per (query token, key/value
+// 640, float32 or bfloat16 storage, float32 arithmetic.  One block per (query token, key/value
 // head, split of the key range); each warp takes query heads of the group in turn, walks the
 // visible keys 32 at a time (one key per lane for q.k, one head dimension per lane for p.v)
 // with a running max and sum, and either writes the output or, with more than one split, a
@@ -15,7 +15,8 @@
 // kernel, p is not rounded to the cache type before p.v, and keys beyond the query are never read.
 #include "common.cuh"
 
-#define ATT_MAX_DPL 8  // head dimensions per lane: hd <= 256
+#define ATT_MAX_DPL 8        // head dimensions per lane: hd <= 256
+#define ATT_MAX_DPL_WIDE 20  // ... of the instance for wider rows: hd <= 640
 
 template <typename T> struct Vec16;
 template <> struct Vec16<float> { static constexpr int N = 4; };
@@ -52,13 +53,13 @@ __device__ __forceinline__ float dot_row<bf16>(const float* __restrict__ q, cons
     return acc;
 }
 
-template <typename T>
+template <typename T, int MAX_DPL>
 __global__ void paged_attention_generic_kernel(
     const T* __restrict__ q, int q_row_stride, const T* __restrict__ k_pages, const T* __restrict__ v_pages,
     T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
     const int* __restrict__ tok_seg, const int* __restrict__ positions, const int* __restrict__ block_table,
     int table_stride, int nh, int nkv, int hd, int page_size, int window, float scale, int n_splits, float softcap,
-    const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks) {
+    const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks, const float* __restrict__ rates) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float q_s[];  // [warps][hd]
@@ -86,10 +87,11 @@ __global__ void paged_attention_generic_kernel(
         for (int d = lane; d < hd; d += 32) qw[d] = to_f32(qp[d]) * scale;
         __syncwarp();
         float m = -INFINITY, l = 0.f;
-        const float slope = slopes ? slopes[h] : 0.f;      // a distance bias: slope * (query position - key position) is taken off
-        float o[ATT_MAX_DPL];
+        // a distance bias: slope * distance, or with a rate slope * ln(1 + rate * distance), is taken off the score
+        const float slope = slopes ? slopes[h] : 0.f, rate = rates ? rates[h] : 0.f;
+        float o[MAX_DPL];
 #pragma unroll
-        for (int j = 0; j < ATT_MAX_DPL; ++j) o[j] = 0.f;
+        for (int j = 0; j < MAX_DPL; ++j) o[j] = 0.f;
 
         for (int n0 = begin; n0 < end; n0 += 32) {
             const int n = n0 + lane;
@@ -101,14 +103,14 @@ __global__ void paged_attention_generic_kernel(
                 row = (((long long)page * nkv + kh) * page_size + (n % page_size)) * hd;
                 s = dot_row<T>(qw, k_pages + row, hd);
                 if (softcap > 0.f) s = softcap * tanhf(s / softcap);     // scores are bounded by +-softcap before the softmax
-                s -= slope * (float)(pos - n);
+                if (slopes) s -= slope * (rates ? log1pf(rate * (float)(pos - n)) : (float)(pos - n));
             }
             const float m_new = fmaxf(m, warp_max(s));
             const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
             const float p = valid ? expf(s - m_new) : 0.f;
             l = l * corr + warp_sum(p);
 #pragma unroll
-            for (int j = 0; j < ATT_MAX_DPL; ++j) o[j] *= corr;
+            for (int j = 0; j < MAX_DPL; ++j) o[j] *= corr;
             m = m_new;
             const int cnt = min(32, end - n0);
             for (int j = 0; j < cnt; ++j) {
@@ -116,7 +118,7 @@ __global__ void paged_attention_generic_kernel(
                 const long long rj = __shfl_sync(0xffffffffu, row, j);
                 const T* vp = v_pages + rj;
 #pragma unroll
-                for (int jj = 0; jj < ATT_MAX_DPL; ++jj) {
+                for (int jj = 0; jj < MAX_DPL; ++jj) {
                     const int d = lane + 32 * jj;
                     if (d < hd) o[jj] += pj * to_f32(vp[d]);
                 }
@@ -128,12 +130,12 @@ __global__ void paged_attention_generic_kernel(
                 const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
                 l = l * corr + expf(sinks[h] - m_new);
 #pragma unroll
-                for (int j = 0; j < ATT_MAX_DPL; ++j) o[j] *= corr;
+                for (int j = 0; j < MAX_DPL; ++j) o[j] *= corr;
             }
             const float inv = l > 0.f ? 1.0f / l : 0.f;
             T* op = out + ((size_t)t * nh + h) * hd;
 #pragma unroll
-            for (int jj = 0; jj < ATT_MAX_DPL; ++jj) {
+            for (int jj = 0; jj < MAX_DPL; ++jj) {
                 const int d = lane + 32 * jj;
                 if (d < hd) op[d] = from_f32<T>(o[jj] * inv);
             }
@@ -141,7 +143,7 @@ __global__ void paged_attention_generic_kernel(
             const size_t slot = ((size_t)t * nh + h) * n_splits + sp;
             float* po = part_o + slot * hd;
 #pragma unroll
-            for (int jj = 0; jj < ATT_MAX_DPL; ++jj) {
+            for (int jj = 0; jj < MAX_DPL; ++jj) {
                 const int d = lane + 32 * jj;
                 if (d < hd) po[d] = o[jj];
             }
@@ -188,9 +190,10 @@ PICO_API int pico_paged_attention_generic(const void* q, int q_row_stride, const
                                           const int* tok_seg, const int* positions, const int* block_table,
                                           int table_stride, int T, int nh, int nkv, int hd, int page_size,
                                           int window, float scale, int n_splits, float softcap, int act_dtype,
-                                          const float* slopes, int chunk, const float* sinks, cudaStream_t stream) {
+                                          const float* slopes, int chunk, const float* sinks, const float* rates,
+                                          cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (hd % 16 != 0 || hd < 16 || hd > 32 * ATT_MAX_DPL) return PICO_ERR_SIZE;
+    if (hd % 16 != 0 || hd < 16 || hd > 32 * ATT_MAX_DPL_WIDE || (rates && !slopes)) return PICO_ERR_SIZE;
     if (nkv <= 0 || nh % nkv != 0 || n_splits < 1 || n_splits > 65535 || nkv > 65535) return PICO_ERR_SIZE;
     if (n_splits > 1 && (!part_o || !part_ml)) return PICO_ERR_SIZE;
     if (chunk < 0) return PICO_ERR_SIZE;
@@ -198,23 +201,23 @@ PICO_API int pico_paged_attention_generic(const void* q, int q_row_stride, const
     const int warps = g < 4 ? g : 4;
     const dim3 grid(T, nkv, n_splits);
     const size_t smem = (size_t)warps * hd * sizeof(float);
+#define LAUNCH_GENERIC(TA, DPL)                                                                                          \
+    pico_launch((paged_attention_generic_kernel<TA, DPL>), dim3(grid), dim3(warps * 32), smem, stream, (const TA*)q,      \
+                q_row_stride, (const TA*)k_pages, (const TA*)v_pages, (TA*)out, part_o, part_ml, tok_seg, positions,      \
+                block_table, table_stride, nh, nkv, hd, page_size, window, scale, n_splits, softcap, slopes, chunk, sinks, rates)
+    const bool wide = hd > 32 * ATT_MAX_DPL;
     if (act_dtype == PICO_F32) {
         if ((q_row_stride % 4) != 0) return PICO_ERR_ALIGN;
-        pico_launch((paged_attention_generic_kernel<float>), dim3(grid), dim3(warps * 32), smem, stream, 
-            (const float*)q, q_row_stride, (const float*)k_pages, (const float*)v_pages, (float*)out, part_o,
-            part_ml, tok_seg, positions, block_table, table_stride, nh, nkv, hd, page_size, window, scale, n_splits, softcap,
-            slopes, chunk, sinks);
+        if (wide) LAUNCH_GENERIC(float, ATT_MAX_DPL_WIDE); else LAUNCH_GENERIC(float, ATT_MAX_DPL);
         if (n_splits > 1)
             pico_launch((attention_combine_kernel<float>), dim3(T * nh), dim3(64), 0, stream, part_o, part_ml, (float*)out, hd, n_splits, sinks, nh);
     } else if (act_dtype == PICO_BF16) {
-        pico_launch((paged_attention_generic_kernel<bf16>), dim3(grid), dim3(warps * 32), smem, stream, 
-            (const bf16*)q, q_row_stride, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out, part_o, part_ml,
-            tok_seg, positions, block_table, table_stride, nh, nkv, hd, page_size, window, scale, n_splits, softcap, slopes, chunk,
-            sinks);
+        if (wide) LAUNCH_GENERIC(bf16, ATT_MAX_DPL_WIDE); else LAUNCH_GENERIC(bf16, ATT_MAX_DPL);
         if (n_splits > 1)
             pico_launch((attention_combine_kernel<bf16>), dim3(T * nh), dim3(64), 0, stream, part_o, part_ml, (bf16*)out, hd, n_splits, sinks, nh);
     } else
         return PICO_ERR_DTYPE;
+#undef LAUNCH_GENERIC
     return pico_launch_status();
 }
 
@@ -278,7 +281,7 @@ PICO_API int pico_paged_attention_noalloc(const void* q, int q_row_stride, const
     float* part_ml = part_o + (size_t)T * nh * n_splits * hd;
     const int rc = pico_paged_attention_generic(q, q_row_stride, k_pages, v_pages, out, part_o, part_ml, tok_seg,
                                                 positions, block_table, table_stride, T, nh, nkv, hd, page_size,
-                                                window, scale, n_splits, 0.f, act_dtype, nullptr, 0, nullptr, stream);
+                                                window, scale, n_splits, 0.f, act_dtype, nullptr, 0, nullptr, nullptr, stream);
     if (rc == PICO_ERR_SIZE) return noalloc_fail(rc, err, err_len, "a size the attention kernels do not take");
     if (rc == PICO_ERR_DTYPE) return noalloc_fail(rc, err, err_len, "act_dtype must be 0 (float32) or 1 (bfloat16)");
     if (rc == PICO_ERR_ALIGN) return noalloc_fail(rc, err, err_len, "q_row_stride must be a multiple of 4 for float32");

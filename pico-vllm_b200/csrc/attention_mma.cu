@@ -119,7 +119,8 @@ __device__ __forceinline__ void pv_tile(float (&o)[HD_MAX / 8][4], const float (
 // ------------------------------------------------------------------------------------------ prefill
 // grid: (tiles of tokens, kv heads, listed segments).  A block takes `tpt` = 64 / g tokens of one
 // segment and the g query heads of one kv head: 64 rows, 16 per warp.
-// EXTRA: a distance bias slope_h * (query position - key position) taken off head h's scores, only
+// EXTRA: a distance bias slope_h * (query position - key position) - with `rates` slope_h * ln(1 + rate_h * distance) - taken
+// off head h's scores, only
 // the keys of the query's own chunk of `chunk` positions (counted from the request's start; 0: all), and a sink, one more
 // term exp(sinks[h]) in the softmax's denominator that has no value (nullptr: none)
 template <int HD_MAX, bool EXTRA>
@@ -129,7 +130,8 @@ paged_prefill_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf1
                          const int* __restrict__ cu_q, const int* __restrict__ positions,
                          const int* __restrict__ block_table, int table_stride, int nh, int nkv, int hd,
                          int page_size, int window, float scale_log2, float cap_log2, float cap_2x,
-                         const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks) {
+                         const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks,
+                         const float* __restrict__ rates) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -173,7 +175,8 @@ paged_prefill_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf1
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     // positions of the two rows this thread holds
     int row_pos[2], row_lo[2];
-    float row_slope[2] = {0.f, 0.f};
+    float row_slope[2] = {0.f, 0.f}, row_rate[2] = {0.f, 0.f};
+    const bool log_bias = EXTRA && rates;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         const int row = warp * 16 + (lane >> 2) + r * 8;
@@ -181,7 +184,8 @@ paged_prefill_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf1
         row_pos[r] = tok < ntok ? pos0 + tok : -1;             // -1: a padding row sees nothing
         row_lo[r] = (window > 0 && row_pos[r] + 1 > window) ? row_pos[r] + 1 - window : 0;
         if (EXTRA && chunk > 0 && row_pos[r] >= 0) row_lo[r] = max(row_lo[r], row_pos[r] / chunk * chunk);
-        if (EXTRA && slopes) row_slope[r] = slopes[kh * g + row - tok * g] * 1.4426950408889634f;
+        if (EXTRA && slopes) row_slope[r] = slopes[kh * g + row - tok * g] * (log_bias ? 1.0f : 1.4426950408889634f);
+        if (log_bias) row_rate[r] = rates[kh * g + row - tok * g];
     }
     // the last key any row of this warp sees: later tiles are skipped by this warp
     const int warp_last_tok = min(ntok - 1, (warp * 16 + 15) / g);
@@ -212,7 +216,9 @@ paged_prefill_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf1
                     const int r = e >> 1;
                     const bool vis = n <= row_pos[r] && n >= row_lo[r];
                     s[j][e] = vis ? pico_score_log2(s[j][e], scale_log2, cap_log2, cap_2x) : -INFINITY;
-                    if (EXTRA && vis) s[j][e] = fmaf(row_slope[r], (float)(n - row_pos[r]), s[j][e]);
+                    if (EXTRA && vis)
+                        s[j][e] = log_bias ? s[j][e] - pico_log_bias(row_slope[r], row_rate[r], (float)(row_pos[r] - n))
+                                           : fmaf(row_slope[r], (float)(n - row_pos[r]), s[j][e]);
                 }
             }
             online_softmax<HD_MAX, MMA_BN / 8>(s, m, l, o);
@@ -247,7 +253,8 @@ paged_decode_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
                         const int* __restrict__ tok_seg, const int* __restrict__ positions,
                         const int* __restrict__ block_table, int table_stride, int nh, int nkv, int hd,
                         int page_size, int window, float scale_log2, int n_splits, float cap_log2, float cap_2x,
-                        const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks) {
+                        const float* __restrict__ slopes, int chunk, const float* __restrict__ sinks,
+                        const float* __restrict__ rates) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -292,12 +299,14 @@ paged_decode_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
 #pragma unroll
     for (int i = 0; i < HD_MAX / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    float row_slope[2] = {0.f, 0.f};
+    float row_slope[2] = {0.f, 0.f}, row_rate[2] = {0.f, 0.f};
+    const bool log_bias = EXTRA && rates;
     if (EXTRA && slopes) {
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             const int row = (lane >> 2) + r * 8;
-            if (row < g) row_slope[r] = slopes[kh * g + row] * 1.4426950408889634f;
+            if (row < g) row_slope[r] = slopes[kh * g + row] * (log_bias ? 1.0f : 1.4426950408889634f);
+            if (row < g && log_bias) row_rate[r] = rates[kh * g + row];
         }
     }
 
@@ -327,7 +336,9 @@ paged_decode_mma_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
                 for (int e = 0; e < 4; ++e) {
                     const int n = w0 + j * 8 + (lane & 3) * 2 + (e & 1);
                     s[j][e] = n < end ? pico_score_log2(s[j][e], scale_log2, cap_log2, cap_2x) : -INFINITY;
-                    if (EXTRA && n < end) s[j][e] = fmaf(row_slope[e >> 1], (float)(n - pos), s[j][e]);
+                    if (EXTRA && n < end)
+                        s[j][e] = log_bias ? s[j][e] - pico_log_bias(row_slope[e >> 1], row_rate[e >> 1], (float)(pos - n))
+                                           : fmaf(row_slope[e >> 1], (float)(n - pos), s[j][e]);
                 }
             online_softmax<HD_MAX, 2>(s, m, l, o);
             pv_tile<HD_MAX, 2>(o, s, v_s + (buf * MMA_BN + warp * 16) * ld, hd, ld, lane);
@@ -448,9 +459,10 @@ PICO_API int pico_paged_prefill_mma(const void* q, int q_row_stride, const void*
                                     void* out, const int* seg_list, int n_segs, const int* cu_q, int max_q_len,
                                     const int* positions, const int* block_table, int table_stride, int nh,
                                     int nkv, int hd, int page_size, int window, float scale, float softcap,
-                                    const float* slopes, int chunk, const float* sinks, cudaStream_t stream) {
+                                    const float* slopes, int chunk, const float* sinks, const float* rates,
+                                    cudaStream_t stream) {
     if (n_segs <= 0 || max_q_len <= 0) return 0;
-    if (chunk < 0) return PICO_ERR_SIZE;
+    if (chunk < 0 || (rates && !slopes)) return PICO_ERR_SIZE;
     const bool extra = slopes || chunk > 0 || sinks;
     if (hd % 16 != 0 || hd < 16 || hd > 256 || nkv <= 0 || nh % nkv != 0) return PICO_ERR_SIZE;
     const int g = nh / nkv;
@@ -467,7 +479,7 @@ PICO_API int pico_paged_prefill_mma(const void* q, int q_row_stride, const void*
         pico_launch((paged_prefill_mma_kernel<HD, X>), dim3(grid), dim3(MMA_THREADS), smem, stream,                 \
             (const bf16*)q, q_row_stride, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out, seg_list, cu_q,   \
             positions, block_table, table_stride, nh, nkv, hd, page_size, window, scale_log2, cap_log2, cap_2x,     \
-            slopes, chunk, sinks);                                                                        \
+            slopes, chunk, sinks, rates);                                                                 \
     } while (0)
 #define LAUNCH_PREFILL(HD) do { if (extra) LAUNCH_PREFILL_X(HD, true); else LAUNCH_PREFILL_X(HD, false); } while (0)
     if (hd <= 64) LAUNCH_PREFILL(64);
@@ -486,9 +498,9 @@ PICO_API int pico_paged_decode_mma(const void* q, int q_row_stride, const void* 
                                    const int* tok_seg, const int* positions, const int* block_table,
                                    int table_stride, int nh, int nkv, int hd, int page_size, int window,
                                    float scale, int n_splits, float softcap, const float* slopes, int chunk,
-                                   const float* sinks, cudaStream_t stream) {
+                                   const float* sinks, const float* rates, cudaStream_t stream) {
     if (n_tok <= 0) return 0;
-    if (chunk < 0) return PICO_ERR_SIZE;
+    if (chunk < 0 || (rates && !slopes)) return PICO_ERR_SIZE;
     const bool extra = slopes || chunk > 0 || sinks;
     if (hd % 16 != 0 || hd < 16 || hd > 256 || nkv <= 0 || nh % nkv != 0) return PICO_ERR_SIZE;
     const int g = nh / nkv;
@@ -505,7 +517,7 @@ PICO_API int pico_paged_decode_mma(const void* q, int q_row_stride, const void* 
         pico_launch((paged_decode_mma_kernel<HD, X>), dim3(grid), dim3(MMA_THREADS), smem, stream,                 \
             (const bf16*)q, q_row_stride, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out, part_o, part_ml, \
             tok_list, tok_seg, positions, block_table, table_stride, nh, nkv, hd, page_size, window, scale_log2,   \
-            n_splits, cap_log2, cap_2x, slopes, chunk, sinks);                                           \
+            n_splits, cap_log2, cap_2x, slopes, chunk, sinks, rates);                                    \
     } while (0)
 #define LAUNCH_DECODE(HD) do { if (extra) LAUNCH_DECODE_X(HD, true); else LAUNCH_DECODE_X(HD, false); } while (0)
     if (hd <= 64) LAUNCH_DECODE(64);

@@ -179,7 +179,8 @@ __device__ __forceinline__ void tca_softmax_sync() { asm volatile("bar.sync 2, 2
 #define TCA_COL_Q 448          // the queries as a tensor-memory operand: 64 columns of bfloat16 pairs at head size 128
 
 // CAP: the scaled scores pass through a soft cap c * tanh(s / c) before the softmax (cap_log2 = c log2 e, cap_2x = 2 scale / c)
-// EXTRA (without CAP): a distance bias slope_h * (query position - key position) taken off head h's scores, only the keys of the query's own chunk of `chunk` positions (counted from the request's start; 0: all), and a sink,
+// EXTRA (without CAP): a distance bias slope_h * (query position - key position) - with `rates` slope_h * ln(1 + rate_h *
+// distance) - taken off head h's scores, only the keys of the query's own chunk of `chunk` positions (counted from the request's start; 0: all), and a sink,
 // one more term exp(sinks[h]) in the softmax's denominator that has no value (nullptr: none)
 template <int HD, bool CAP, bool EXTRA>      // head size, a multiple of 64 up to 128
 __global__ void __launch_bounds__(TCA_THREADS)
@@ -190,7 +191,7 @@ paged_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
                              int nh, int nkv, int page_size, int window, float scale_log2, float cap_log2, float cap_2x,
                              float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                              size_t n_rows, int n_parts, int split_min, const float* __restrict__ slopes, int chunk,
-                             const float* __restrict__ sinks) {
+                             const float* __restrict__ sinks, const float* __restrict__ rates) {
     pdl_launch_dependents();
     extern __shared__ unsigned char tca_dyn[];
     constexpr int NH = HD / 64;                              // 64-dim blocks of a head
@@ -386,7 +387,9 @@ paged_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
         const int row_pos = row_ok ? pos0 + tok : -1;
         int row_lo = (window > 0 && row_pos + 1 > window) ? row_pos + 1 - window : 0;
         if (EXTRA && chunk > 0 && row_ok) row_lo = max(row_lo, row_pos / chunk * chunk);
-        const float slope2 = (EXTRA && slopes) ? slopes[kh * g + head] * 1.4426950408889634f : 0.f;     // log2 units
+        const bool log_bias = EXTRA && rates;
+        const float slope2 = (EXTRA && slopes) ? slopes[kh * g + head] * (log_bias ? 1.0f : 1.4426950408889634f) : 0.f;     // log2 units
+        const float rate = log_bias ? rates[kh * g + head] : 0.f;
         const uint32_t lane_off = (uint32_t)(qtr * 32) << 16;
         const uint32_t tmem_s = tmem_base + TCA_COL_S + pipe * TCA_BN + lane_off;
         const uint32_t tmem_p = tmem_base + TCA_COL_P + pipe * (TCA_BN / 2) + lane_off;
@@ -442,7 +445,20 @@ paged_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
                     if (!(n <= row_pos && n >= row_lo)) sv[c] = 0xff800000u;     // -inf
                 }
             }
-            if (EXTRA) {     // scores in log2 units with the distance bias taken off; a hidden key stays at -inf
+            if (EXTRA && log_bias) {     // slope log2(1 + rate * distance) taken off, two keys at a time; what lies ahead of the query is hidden
+                const float d0 = (float)(row_pos - n0);
+                const uint64_t d2 = tca_pack(d0, d0), rate2 = tca_pack(rate, rate), one = tca_pack(1.0f, 1.0f);
+                const uint64_t neg_slope2 = tca_pack(-slope2, -slope2);
+#pragma unroll
+                for (int c = 0; c < 64; c += 2) {
+                    float a0, a1, y0, y1;
+                    tca_unpack(tca_fma2(rate2, tca_add2(d2, tca_pack(-(float)c, -(float)(c + 1))), one), a0, a1);
+                    const uint64_t lg = tca_pack(__log2f(fmaxf(a0, 1e-30f)), __log2f(fmaxf(a1, 1e-30f)));
+                    tca_unpack(tca_fma2(tca_pack(__uint_as_float(sv[c]), __uint_as_float(sv[c + 1])), scale2, tca_fma2(neg_slope2, lg, 0ull)), y0, y1);
+                    sv[c] = __float_as_uint(y0);
+                    sv[c + 1] = __float_as_uint(y1);
+                }
+            } else if (EXTRA) {     // scores in log2 units with the distance bias taken off; a hidden key stays at -inf
                 const float base = fmaf(slope2, (float)(n0 - row_pos), 0.f);
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
@@ -736,7 +752,7 @@ PICO_API int pico_paged_prefill_tcgen05(const void* k_map, const void* v_map, co
                                         const int* positions, const int* block_table, int table_stride, int nh, int nkv,
                                         int hd, int page_size, int window, float scale, int pair_min_keys, float* scratch,
                                         int n_tokens, int* counters, int n_counters, float softcap, const float* slopes,
-                                        int chunk, const float* sinks, cudaStream_t stream) {
+                                        int chunk, const float* sinks, const float* rates, cudaStream_t stream) {
     if (n_segs <= 0 || max_q_len <= 0) return 0;
     if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv != 0) return PICO_ERR_SIZE;
     const int g = nh / nkv;
@@ -744,7 +760,7 @@ PICO_API int pico_paged_prefill_tcgen05(const void* k_map, const void* v_map, co
     if (page_size < 8 || TCA_BN % page_size != 0) return PICO_ERR_SIZE;
     if (q_row_stride % 8 != 0) return PICO_ERR_ALIGN;
     const bool extra = slopes || chunk > 0 || sinks;
-    if (chunk < 0 || (extra && softcap > 0.f)) return PICO_ERR_SIZE;       // the bias is not built together with the cap
+    if (chunk < 0 || (extra && softcap > 0.f) || (rates && !slopes)) return PICO_ERR_SIZE;       // the bias is not built together with the cap
     if (extra) pair_min_keys = 0;                                          // nor with tiles shared by two blocks
     const int tpt = TCA_BM / g;
     const int n_qt = (max_q_len + tpt - 1) / tpt;
@@ -765,7 +781,7 @@ PICO_API int pico_paged_prefill_tcgen05(const void* k_map, const void* v_map, co
         cudaFuncSetAttribute(paged_prefill_tcgen05_kernel<HD, CAP, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         pico_launch((paged_prefill_tcgen05_kernel<HD, CAP, EXTRA>), grid, dim3(TCA_THREADS), smem, stream, km, vm, (const bf16*)q, \
                     q_row_stride, (bf16*)out, seg_list, cu_q, positions, block_table, table_stride, nh, nkv, page_size,  \
-                    window, scale_log2, cap_log2, cap_2x, part_o, part_ml, counters, n_rows, n_parts, split_min, slopes, chunk, sinks); \
+                    window, scale_log2, cap_log2, cap_2x, part_o, part_ml, counters, n_rows, n_parts, split_min, slopes, chunk, sinks, rates); \
     } while (0)
     if (hd == 64) { if (extra) LAUNCH_TCA(64, false, true); else if (cap_log2 > 0.f) LAUNCH_TCA(64, true, false); else LAUNCH_TCA(64, false, false); }
     else { if (extra) LAUNCH_TCA(128, false, true); else if (cap_log2 > 0.f) LAUNCH_TCA(128, true, false); else LAUNCH_TCA(128, false, false); }

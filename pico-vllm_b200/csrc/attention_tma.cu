@@ -98,15 +98,19 @@ __device__ __forceinline__ uint32_t tile_off(int key, int dim, int page_size) {
 // with stage s.
 // CW consumer warps in groups of four: group i takes tiles i, i + CW/4, ... (a group multiplies one tile,
 // 16 cache positions per warp); one group is what the launcher uses.
-// CAP: scores pass through a soft cap (cap_log2, cap_2x as for pico_score_log2); without it the kernel is what it was
-template <int HD, int TMA_STAGES, int CW, int NT, bool CAP>     // head size 64 or 128; stages; consumer warps (4 or 8); 8-head tiles (g <= 8 NT)
+// MODE: TMA_PLAIN; TMA_CAP - scores pass through a soft cap (cap_log2, cap_2x as for pico_score_log2); TMA_EXTRA - a distance
+// bias (slopes, with rates logarithmic, as in attention_mma.cu) is taken off the scores and / or the softmax has a sink
+// (sinks[h]: one more term of the denominator, which joins the first part of a token's key range)
+enum { TMA_PLAIN = 0, TMA_CAP = 1, TMA_EXTRA = 2 };
+template <int HD, int TMA_STAGES, int CW, int NT, int MODE>     // head size 64 or 128; stages; consumer warps (4 or 8); 8-head tiles (g <= 8 NT)
 __global__ void __launch_bounds__((CW + 1) * 32)
 paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                         const bf16* __restrict__ q, int q_row_stride, bf16* __restrict__ out,
                         float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ tok_list,
                         const int* __restrict__ tok_seg, const int* __restrict__ positions,
                         const int* __restrict__ block_table, int table_stride, int nh, int nkv, int page_size,
-                        int window, float scale_log2, int n_splits, int cluster_reduce, int kv_same, float cap_log2, float cap_2x) {
+                        int window, float scale_log2, int n_splits, int cluster_reduce, int kv_same, float cap_log2, float cap_2x,
+                        const float* __restrict__ slopes, const float* __restrict__ sinks, const float* __restrict__ rates) {
     // kv_same: keys and values are one tensor (a cached latent that serves as both): only the key tile is copied and
     // the p.v product reads it too - the two maps give tiles of the same layout
     pdl_launch_dependents();
@@ -246,6 +250,18 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
         k_off[i] = tile_off<HD>(kw + a_row, i * 16 + a_col, page_size);
         v_off[i] = tile_off<HD>(kw + v_row, i * 16 + v_col, page_size);
     }
+    constexpr bool CAP = MODE == TMA_CAP, EXTRA = MODE == TMA_EXTRA;
+    const bool log_bias = EXTRA && rates;
+    float sl[NT][2], rt[NT][2];                                  // bias of the thread's head columns
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int row = nt * 8 + (lane & 3) * 2 + h;
+            const bool have = EXTRA && slopes && row < g;
+            sl[nt][h] = have ? slopes[kh * g + row] * (log_bias ? 1.0f : 1.4426950408889634f) : 0.f;
+            rt[nt][h] = have && log_bias ? rates[kh * g + row] : 0.f;
+        }
     for (int it = grp; it < ntiles; it += NG) {
         const int s = it % TMA_STAGES;
         const int n0 = (t_begin + it) * MMA_BN;
@@ -283,6 +299,10 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
                 for (int e = 0; e < 4; ++e) {
                     const float v = (sc[nt][0][e] + sc[nt][1][e]) + (sc[nt][2][e] + sc[nt][3][e]);
                     x[e] = ((e < 2) ? vis_a : vis_b) ? (CAP ? pico_score_log2(v, scale_log2, cap_log2, cap_2x) : v * scale_log2) : -INFINITY;
+                    if (EXTRA && slopes) {                       // a hidden key stays at -inf
+                        const float dist = (float)max(pos - ((e < 2) ? key_a : key_b), 0);
+                        x[e] -= log_bias ? pico_log_bias(sl[nt][e & 1], rt[nt][e & 1], dist) : sl[nt][e & 1] * dist;
+                    }
                 }
                 float p[4];
 #pragma unroll
@@ -392,6 +412,13 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
             }
         }
         const int h = kh * g + row;
+        if (EXTRA && sinks && sp == 0) {          // the sink joins the first part: one more term of its denominator
+            const float sk = sinks[h] * 1.4426950408889634f, mm = fmaxf(M, sk);
+            const float f = M == -INFINITY ? 0.f : fast_exp2(M - mm);
+            L = L * f + fast_exp2(sk - mm);
+            acc *= f;
+            M = mm;
+        }
         if (n_splits == 1) {
             out[((size_t)t * nh + h) * HD + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
         } else if (cluster_reduce) {
@@ -479,14 +506,14 @@ int pico_launch_decode_combine(const float* part_o, const float* part_ml, void* 
                                int nh, int hd, int n_splits, cudaStream_t stream);
 
 // Can clusters of `size` blocks of the decode kernel run here?  (Asked once per configuration.)
-template <int HD, int ST, int CW, int NT, bool CAP>
+template <int HD, int ST, int CW, int NT, int MODE>
 static bool tma_cluster_query(int size, size_t smem) {
-    if (size > 8 && cudaFuncSetAttribute(paged_decode_tma_kernel<HD, ST, CW, NT, CAP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) !=
+    if (size > 8 && cudaFuncSetAttribute(paged_decode_tma_kernel<HD, ST, CW, NT, MODE>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) !=
                         cudaSuccess) {
         cudaGetLastError();
         return false;
     }
-    cudaFuncSetAttribute(paged_decode_tma_kernel<HD, ST, CW, NT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(paged_decode_tma_kernel<HD, ST, CW, NT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(size, 1, 1);
     cfg.blockDim = dim3((CW + 1) * 32);
@@ -499,22 +526,22 @@ static bool tma_cluster_query(int size, size_t smem) {
     cfg.attrs = attr;
     cfg.numAttrs = 1;
     int n = 0;
-    if (cudaOccupancyMaxActiveClusters(&n, paged_decode_tma_kernel<HD, ST, CW, NT, CAP>, &cfg) != cudaSuccess) {
+    if (cudaOccupancyMaxActiveClusters(&n, paged_decode_tma_kernel<HD, ST, CW, NT, MODE>, &cfg) != cudaSuccess) {
         cudaGetLastError();
         return false;
     }
     return n > 0;
 }
-template <bool CAP>
+template <int MODE>
 static bool tma_cluster_ok(int hd, int size, int nt, size_t smem) {
-    static int cache[2][2][5];      // [hd 64/128][head tiles - 1][log2 size]: 0 unknown, 1 yes, 2 no (one table per CAP)
+    static int cache[2][2][5];      // [hd 64/128][head tiles - 1][log2 size]: 0 unknown, 1 yes, 2 no (one table per MODE)
     int lg = 0;
     while ((1 << lg) < size) ++lg;
     int& c = cache[hd == 128 ? 1 : 0][nt - 1][lg];
     if (c == 0) {
         bool ok;
-        if (hd == 128) ok = nt == 1 ? tma_cluster_query<128, TMA_STAGES_MANY, 4, 1, CAP>(size, smem) : tma_cluster_query<128, TMA_STAGES_MANY, 4, 2, CAP>(size, smem);
-        else ok = nt == 1 ? tma_cluster_query<64, TMA_STAGES_MANY, 4, 1, CAP>(size, smem) : tma_cluster_query<64, TMA_STAGES_MANY, 4, 2, CAP>(size, smem);
+        if (hd == 128) ok = nt == 1 ? tma_cluster_query<128, TMA_STAGES_MANY, 4, 1, MODE>(size, smem) : tma_cluster_query<128, TMA_STAGES_MANY, 4, 2, MODE>(size, smem);
+        else ok = nt == 1 ? tma_cluster_query<64, TMA_STAGES_MANY, 4, 1, MODE>(size, smem) : tma_cluster_query<64, TMA_STAGES_MANY, 4, 2, MODE>(size, smem);
         c = ok ? 1 : 2;
     }
     return c == 1;
@@ -526,8 +553,11 @@ PICO_API int pico_paged_decode_tma(const void* k_map, const void* v_map, const v
                                    float* part_o, float* part_ml, const int* tok_list, int n_tok, const int* tok_seg,
                                    const int* positions, const int* block_table, int table_stride, int nh, int nkv,
                                    int hd, int page_size, int window, float scale, int n_splits, int kv_same,
-                                   float softcap, cudaStream_t stream) {
+                                   float softcap, const float* slopes, const float* sinks, const float* rates,
+                                   cudaStream_t stream) {
     if (n_tok <= 0) return 0;
+    const bool extra = slopes || sinks;
+    if ((extra && softcap > 0.f) || (rates && !slopes)) return PICO_ERR_SIZE;
     if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv != 0) return PICO_ERR_SIZE;
     const int g = nh / nkv;
     if (g > 16 || nkv > 65535 || n_tok > 65535 || n_splits < 1 || n_splits > 64) return PICO_ERR_SIZE;
@@ -549,20 +579,23 @@ PICO_API int pico_paged_decode_tma(const void* k_map, const void* v_map, const v
     // 2, 4, 8 or 16 splits: the splits of one (token, kv head) run as one thread-block cluster and are
     // added through distributed shared memory; otherwise through scratch and the combine kernel
     int cluster = 0;
-    if (n_splits == 2 || n_splits == 4 || n_splits == 8 || n_splits == 16) cluster = (cap_log2 > 0.f ? tma_cluster_ok<true>(hd, n_splits, nt, smem) : tma_cluster_ok<false>(hd, n_splits, nt, smem)) ? 1 : 0;
+    if (n_splits == 2 || n_splits == 4 || n_splits == 8 || n_splits == 16) 
+        cluster = (extra ? tma_cluster_ok<TMA_EXTRA>(hd, n_splits, nt, smem) : cap_log2 > 0.f ? tma_cluster_ok<TMA_CAP>(hd, n_splits, nt, smem)
+                                                                             : tma_cluster_ok<TMA_PLAIN>(hd, n_splits, nt, smem)) ? 1 : 0;
     if (n_splits > 1 && !cluster && (!part_o || !part_ml)) return PICO_ERR_SIZE;
-#define LAUNCH_TMA_C(HD, NT, CAP)                                                                                       \
+#define LAUNCH_TMA_C(HD, NT, MODE)                                                                                      \
     do {                                                                                                                \
-        cudaFuncSetAttribute(paged_decode_tma_kernel<HD, TMA_STAGES_MANY, 4, NT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+        cudaFuncSetAttribute(paged_decode_tma_kernel<HD, TMA_STAGES_MANY, 4, NT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                              (int)smem);                                                                                \
-        pico_launch_cluster((paged_decode_tma_kernel<HD, TMA_STAGES_MANY, 4, NT, CAP>), grid, dim3(5 * 32), smem, stream, \
+        pico_launch_cluster((paged_decode_tma_kernel<HD, TMA_STAGES_MANY, 4, NT, MODE>), grid, dim3(5 * 32), smem, stream, \
                             cluster ? n_splits : 1, km, vm, (const bf16*)q, q_row_stride, (bf16*)out, part_o,           \
                             part_ml, tok_list, tok_seg, positions, block_table, table_stride, nh, nkv, page_size,       \
-                            window, scale_log2, n_splits, cluster, kv_same, cap_log2, cap_2x);                          \
+                            window, scale_log2, n_splits, cluster, kv_same, cap_log2, cap_2x, slopes, sinks, rates);    \
     } while (0)
 #define LAUNCH_TMA(HD, NT)                                                                                              \
     do {                                                                                                                \
-        if (cap_log2 > 0.f) LAUNCH_TMA_C(HD, NT, true); else LAUNCH_TMA_C(HD, NT, false);                               \
+        if (extra) LAUNCH_TMA_C(HD, NT, TMA_EXTRA);                                                                     \
+        else if (cap_log2 > 0.f) LAUNCH_TMA_C(HD, NT, TMA_CAP); else LAUNCH_TMA_C(HD, NT, TMA_PLAIN);                   \
     } while (0)
     if (hd == 64) {
         if (nt == 1) LAUNCH_TMA(64, 1); else LAUNCH_TMA(64, 2);

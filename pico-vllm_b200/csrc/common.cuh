@@ -73,6 +73,12 @@ __device__ __forceinline__ float pico_score_log2(float raw, float scale_log2, fl
     return raw * scale_log2;
 }
 
+// What a distance bias takes off a score, in log2 units.  Linear: slope2 * distance with slope2 = slope * log2(e).  With a
+// rate: slope * ln(1 + rate * distance) * log2(e) = slope * log2(1 + rate * distance).
+__device__ __forceinline__ float pico_log_bias(float slope, float rate, float distance) {
+    return slope * __log2f(fmaxf(fmaf(rate, distance, 1.0f), 1e-30f));
+}
+
 static inline int pico_launch_status() { return (int)cudaGetLastError(); }
 
 // Multiprocessors of the current device (asked once per device; grids are sized from it).

@@ -31,7 +31,8 @@
 #define TP_THREADS 192
 #define TP_WAIT_LIMIT (1 << 14)      // polls of a barrier (some microseconds each) before a thread gives up
 
-enum { TP_STORE = 0, TP_RESIDUAL = 1, TP_SWIGLU = 2 };
+enum { TP_STORE = 0, TP_RESIDUAL = 1, TP_SWIGLU = 2, TP_CAPPED = 3 };
+__host__ __device__ constexpr bool tp_is_glu(int epi) { return epi == TP_SWIGLU || epi == TP_CAPPED; }
 
 __device__ int g_tp_status = 0;
 PICO_API int pico_tp_status(int* out) {
@@ -108,6 +109,7 @@ struct TpArgs {
     int M, N, K;              // N: rows of w (SWIGLU: 2 * I)
     bf16* out;                // STORE: [M, N]; SWIGLU: [M, N / 2]
     float* resid;             // RESIDUAL: [M, N]
+    float limit;              // CAPPED: as SWIGLU with g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
 };
 
 __device__ __forceinline__ void tp_st32(void* p, const uint32_t (&r)[8]) {      // one 32-byte store (a whole sector)
@@ -124,6 +126,17 @@ __device__ __forceinline__ float tp_silu_mul(float g, float u) {
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(g * -1.4426950408889634f));
     asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.0f + e));
     return g * r * u;
+}
+__device__ __forceinline__ float tp_capped_mul(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(g * (-1.702f * 1.4426950408889634f)));
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.0f + e));
+    return g * r * (u + 1.0f);
+}
+template <int EPI> __device__ __forceinline__ float tp_glu(float g, float u, float limit) {
+    return EPI == TP_CAPPED ? tp_capped_mul(g, u, limit) : tp_silu_mul(g, u);
 }
 __device__ __forceinline__ uint32_t tp_pack(float a, float b) {
     __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -146,7 +159,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid
     constexpr int ROWS = MB * TP_BM;                           // rows of x per block
     constexpr int NBUF = MB == 1 ? 2 : 1;                      // accumulator buffers (of MB accumulators each)
     constexpr int A_BLOCK = TP_BM * TP_BK * 2, A_BYTES = MB * A_BLOCK, B_BYTES = (BN / 2) * TP_BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
-    constexpr int COLS = EPI == TP_SWIGLU ? BN / 2 : BN;       // output columns of a tile
+    constexpr int COLS = tp_is_glu(EPI) ? BN / 2 : BN;       // output columns of a tile
     constexpr int TMEM_COLS = 512;
     uint64_t* full = reinterpret_cast<uint64_t*>(smem + STAGES * STAGE_BYTES);      // used in block 0: both blocks' copies landed
     uint64_t* empty = full + STAGES;                           // the products have read the stage (both blocks)
@@ -189,7 +202,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid
             int step = 0;
             for (int t = pair; t < total_tiles && !*abort_s; t += n_pairs) {
                 const int m0 = (t % m_tiles) * 2 * ROWS + (int)rank * ROWS, n0 = (t / m_tiles) * COLS;
-                const int w_row = EPI == TP_SWIGLU ? (rank ? p.N / 2 + n0 : n0) : n0 + (int)rank * (BN / 2);
+                const int w_row = tp_is_glu(EPI) ? (rank ? p.N / 2 + n0 : n0) : n0 + (int)rank * (BN / 2);
                 for (int kb = 0; kb < nkb; ++kb, ++step) {
                     const int s = step % STAGES;
                     if (step >= STAGES && !tp_wait(empty + s, ((step / STAGES) - 1) & 1)) {
@@ -256,7 +269,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid
             if (__any_sync(0xffffffffu, !ok || *abort_s != 0)) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const uint32_t taddr = tmem_base + (buf * MB + j) * BN + ((uint32_t)(q * 32) << 16);
-            if (EPI == TP_SWIGLU) {
+            if (tp_is_glu(EPI)) {
                 const int I = p.N / 2;
                 const bool wide = (I & 15) == 0;               // rows of out start on 32 bytes
 #pragma unroll 1
@@ -272,8 +285,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid
                             uint32_t pk[8];
 #pragma unroll
                             for (int e = 0; e < 16; e += 2)
-                                pk[e / 2] = tp_pack(tp_silu_mul(__uint_as_float(g[i + e]), __uint_as_float(u[i + e])),
-                                                    tp_silu_mul(__uint_as_float(g[i + e + 1]), __uint_as_float(u[i + e + 1])));
+                                pk[e / 2] = tp_pack(tp_glu<EPI>(__uint_as_float(g[i + e]), __uint_as_float(u[i + e]), p.limit),
+                                                    tp_glu<EPI>(__uint_as_float(g[i + e + 1]), __uint_as_float(u[i + e + 1]), p.limit));
                             if (wide && n0 + c + i + 16 <= I) {
                                 tp_st32(dst + i, pk);
                             } else {
@@ -402,8 +415,8 @@ static int tp_launch(const void* x, int ldx, const void* w, const TpArgs& a, cud
     if (rc) return rc;
     const size_t smem = (size_t)STAGES * STAGE_BYTES + (2 * STAGES + 4) * 8 + 16 + 1024;
     cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<BN, EPI, STAGES, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    const int n_out = EPI == TP_SWIGLU ? a.N / 2 : a.N;
-    const int cols = EPI == TP_SWIGLU ? BN / 2 : BN;
+    const int n_out = tp_is_glu(EPI) ? a.N / 2 : a.N;
+    const int cols = tp_is_glu(EPI) ? BN / 2 : BN;
     const int n_tiles = (n_out + cols - 1) / cols, m_tiles = (a.M + 2 * MB * TP_BM - 1) / (2 * MB * TP_BM);
     const int max_pairs = tp_num_sms() / 2;
     const int pairs = n_tiles * m_tiles < max_pairs ? n_tiles * m_tiles : max_pairs;
@@ -437,23 +450,25 @@ static void tp_pick(int M, int n_out, bool swiglu, int force_mb, int& bn_out, in
 }
 
 // epi: 0 = out[M, N] = x w^T (bfloat16); 1 = resid[M, N] (float32) += x w^T; 2 = out[M, N/2] =
-// silu(x wg^T) * (x wu^T) with w = [wg; wu].  x: [M, K] bfloat16 with row stride ldx; w: [N, K] contiguous.
+// silu(x wg^T) * (x wu^T) with w = [wg; wu]; 3 = the same with the capped form of the two products (limit > 0).  x: [M, K] bfloat16 with row stride ldx; w: [N, K] contiguous.
 // rows_per_pair: 0 = chosen here, 256 or 512.
 PICO_API int pico_gemm_tcgen05_pair(const void* x, int ldx, const void* w, void* out, float* resid, int M, int N, int K,
-                                    int epi, int rows_per_pair, cudaStream_t stream) {
+                                    int epi, int rows_per_pair, float limit, cudaStream_t stream) {
     if (M < 1 || N < 16 || K < 16 || K % 8 != 0 || ldx % 8 != 0) return PICO_ERR_SIZE;
-    if (epi == TP_SWIGLU && (N % 2 != 0 || (N / 2) % 8 != 0)) return PICO_ERR_SIZE;
-    if (epi != TP_SWIGLU && N % 8 != 0) return PICO_ERR_SIZE;
+    if (epi == TP_CAPPED && !(limit > 0.f)) return PICO_ERR_SIZE;
+    if (tp_is_glu(epi) && (N % 2 != 0 || (N / 2) % 8 != 0)) return PICO_ERR_SIZE;
+    if (!tp_is_glu(epi) && N % 8 != 0) return PICO_ERR_SIZE;
     if (rows_per_pair != 0 && rows_per_pair != 256 && rows_per_pair != 512) return PICO_ERR_SIZE;
     TpArgs a;
-    a.M = M; a.N = N; a.K = K; a.out = (bf16*)out; a.resid = resid;
+    a.M = M; a.N = N; a.K = K; a.out = (bf16*)out; a.resid = resid; a.limit = limit;
     int bn = 256, mb = 1;
-    tp_pick(M, epi == TP_SWIGLU ? N / 2 : N, epi == TP_SWIGLU, rows_per_pair / 256, bn, mb);
+    tp_pick(M, tp_is_glu(epi) ? N / 2 : N, tp_is_glu(epi), rows_per_pair / 256, bn, mb);
 #define TP_CASE(BN, MB)                                                                       \
     if (bn == BN && mb == MB) {                                                               \
         if (epi == TP_STORE) return tp_launch<BN, TP_STORE, MB>(x, ldx, w, a, stream);        \
         if (epi == TP_RESIDUAL) return tp_launch<BN, TP_RESIDUAL, MB>(x, ldx, w, a, stream);  \
         if (epi == TP_SWIGLU) return tp_launch<BN, TP_SWIGLU, MB>(x, ldx, w, a, stream);      \
+        if (epi == TP_CAPPED) return tp_launch<BN, TP_CAPPED, MB>(x, ldx, w, a, stream);      \
     }
     TP_CASE(256, 2)
     TP_CASE(256, 1)

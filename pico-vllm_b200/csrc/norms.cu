@@ -5,7 +5,8 @@
 //   x  = x + d'               (float32 residual stream, written back unless rows are picked)
 //   y  = N(x)                 (optional; the same two kinds)
 //
-// RMS:      u / sqrt(mean(u^2) + eps) * w
+// RMS:      u / sqrt(mean(u^2) + eps) * w; with `groups` > 1 the row is that many equal runs of neighbours, each divided by
+//           its own root mean square (w covers the whole row)
 // centred:  (u - mean u) / sqrt(mean((u - mean u)^2) + eps) * w     (two passes over the row held in
 //           shared memory: the mean first, then the mean of the squared deviations)
 // All arithmetic in float32; d and y are in the activation type.
@@ -40,8 +41,37 @@ template <> struct Row4<bf16> {
 // i = thread, thread + threads, ...), so loops over the row need no barrier between them.
 template <bool VEC>
 __device__ __forceinline__ void norm_row_inplace(float* vals, int H, int kind, const float* __restrict__ w, float eps,
-                                                 float* scratch) {
+                                                 float* scratch, int groups) {
     const int n = VEC ? H >> 2 : H;
+    if (groups > 1) {       // a root mean square per group; with VEC a vector lies within one group
+        const int gn = n / groups;
+        for (int g = 0; g < groups; ++g) {
+            float gs = 0.f;
+            const int lo = g * gn, hi = lo + gn;
+            for (int i = threadIdx.x; i < hi; i += blockDim.x) {
+                if (i < lo) continue;
+                if (VEC) {
+                    const float4 v = *reinterpret_cast<const float4*>(vals + 4 * i);
+                    gs += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+                } else {
+                    gs += vals[i] * vals[i];
+                }
+            }
+            const float ginv = 1.0f / sqrtf(block_sum(gs, scratch) / (float)(H / groups) + eps);
+            for (int i = threadIdx.x; i < hi; i += blockDim.x) {
+                if (i < lo) continue;
+                if (VEC) {
+                    float4 v = *reinterpret_cast<const float4*>(vals + 4 * i);
+                    const float4 gw = w ? *reinterpret_cast<const float4*>(w + 4 * i) : make_float4(1.f, 1.f, 1.f, 1.f);
+                    v.x *= ginv * gw.x; v.y *= ginv * gw.y; v.z *= ginv * gw.z; v.w *= ginv * gw.w;
+                    *reinterpret_cast<float4*>(vals + 4 * i) = v;
+                } else {
+                    vals[i] *= ginv * (w ? w[i] : 1.f);
+                }
+            }
+        }
+        return;
+    }
     float mean = 0.f;
     if (kind == NORM_CENTRED) {
         float s = 0.f;
@@ -91,7 +121,7 @@ template <typename TA, bool VEC>
 __global__ void post_add_norm_kernel(float* __restrict__ x, const TA* __restrict__ delta,
                                      const float* __restrict__ post_w, int post_kind, float post_eps,
                                      const float* __restrict__ w, int kind, float eps, TA* __restrict__ out,
-                                     const int* __restrict__ rows, int H) {
+                                     const int* __restrict__ rows, int H, int post_groups, int groups) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) float vals[];  // H floats, then 33 of scratch
@@ -105,7 +135,7 @@ __global__ void post_add_norm_kernel(float* __restrict__ x, const TA* __restrict
             if (VEC) *reinterpret_cast<float4*>(vals + 4 * i) = Row4<TA>::load(delta + src + 4 * i);
             else vals[i] = to_f32(delta[src + i]);
         }
-        if (post_kind != NORM_NONE) norm_row_inplace<VEC>(vals, H, post_kind, post_w, post_eps, scratch);
+        if (post_kind != NORM_NONE) norm_row_inplace<VEC>(vals, H, post_kind, post_w, post_eps, scratch, post_groups);
 #pragma unroll 4
         for (int i = threadIdx.x; i < n; i += blockDim.x) {
             if (VEC) {
@@ -132,7 +162,7 @@ __global__ void post_add_norm_kernel(float* __restrict__ x, const TA* __restrict
         }
     }
     if (!out || kind == NORM_NONE) return;
-    if (kind != NORM_COPY) norm_row_inplace<VEC>(vals, H, kind, w, eps, scratch);
+    if (kind != NORM_COPY) norm_row_inplace<VEC>(vals, H, kind, w, eps, scratch, groups);
     else __syncthreads();
     TA* dst = out + (size_t)r * H;
 #pragma unroll 4
@@ -145,9 +175,36 @@ __global__ void post_add_norm_kernel(float* __restrict__ x, const TA* __restrict
 // The same work with a warp per row and the row in registers (H a multiple of 4, at most 128 * VPL elements): every
 // load of a row - what is added and the stream - is issued before anything is waited for, the sums
 // go through shuffles, and nothing passes through shared memory or a block barrier.  Four rows a block.
-template <int VPL>
+// GROUPED: `groups` equal runs of H / groups elements (a multiple of 4), a root mean square each.
+template <int VPL, bool GROUPED>
 __device__ __forceinline__ void norm_regs(float4 (&v)[VPL], const float* __restrict__ w, int n4, int lane, int H, int kind,
-                                          float eps) {
+                                          float eps, int groups) {
+    if (GROUPED && groups > 1) {
+        const int gn = n4 / groups;
+        for (int g = 0; g < groups; ++g) {
+            const int lo = g * gn, hi = lo + gn;
+            float gs = 0.f;
+#pragma unroll
+            for (int k = 0; k < VPL; ++k) {
+                const int i = lane + 32 * k;
+                if (i >= lo && i < hi) gs += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+            }
+            const float ginv = 1.0f / sqrtf(warp_sum(gs) / (float)(4 * gn) + eps);
+#pragma unroll
+            for (int k = 0; k < VPL; ++k) {
+                const int i = lane + 32 * k;
+                if (i >= lo && i < hi) { v[k].x *= ginv; v[k].y *= ginv; v[k].z *= ginv; v[k].w *= ginv; }
+            }
+        }
+        if (!w) return;
+#pragma unroll
+        for (int k = 0; k < VPL; ++k)
+            if (lane + 32 * k < n4) {
+                const float4 g = *reinterpret_cast<const float4*>(w + 4 * (lane + 32 * k));
+                v[k].x *= g.x; v[k].y *= g.y; v[k].z *= g.z; v[k].w *= g.w;
+            }
+        return;
+    }
     float mean = 0.f;
     if (kind == NORM_CENTRED) {
         float s = 0.f;
@@ -175,12 +232,13 @@ __device__ __forceinline__ void norm_regs(float4 (&v)[VPL], const float* __restr
     }
 }
 
-template <typename TA, int VPL>
+template <typename TA, int VPL, bool GROUPED>
 __global__ void __launch_bounds__(128) post_add_norm_warp_kernel(float* __restrict__ x, const TA* __restrict__ delta,
                                                                  const float* __restrict__ post_w, int post_kind,
                                                                  float post_eps, const float* __restrict__ w, int kind,
                                                                  float eps, TA* __restrict__ out,
-                                                                 const int* __restrict__ rows, int R, int H) {
+                                                                 const int* __restrict__ rows, int R, int H, int post_groups,
+                                                                 int groups) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -199,27 +257,27 @@ __global__ void __launch_bounds__(128) post_add_norm_warp_kernel(float* __restri
         d[k] = ok && delta ? Row4<TA>::load(delta + src + 4 * i) : zero;
         a[k] = ok ? *reinterpret_cast<const float4*>(x + src + 4 * i) : zero;
     }
-    if (norm_in) norm_regs<VPL>(d, post_w, n4, lane, H, post_kind, post_eps);
+    if (norm_in) norm_regs<VPL, GROUPED>(d, post_w, n4, lane, H, post_kind, post_eps, post_groups);
 #pragma unroll
     for (int k = 0; k < VPL; ++k) {
         a[k].x += d[k].x; a[k].y += d[k].y; a[k].z += d[k].z; a[k].w += d[k].w;
         if (delta && !rows && lane + 32 * k < n4) *reinterpret_cast<float4*>(x + src + 4 * (lane + 32 * k)) = a[k];
     }
     if (!norm_out) return;
-    if (kind != NORM_COPY) norm_regs<VPL>(a, w, n4, lane, H, kind, eps);
+    if (kind != NORM_COPY) norm_regs<VPL, GROUPED>(a, w, n4, lane, H, kind, eps, groups);
     TA* dst = out + (size_t)r * H;
 #pragma unroll
     for (int k = 0; k < VPL; ++k)
         if (lane + 32 * k < n4) Row4<TA>::store(dst + 4 * (lane + 32 * k), a[k]);
 }
 
-template <typename TA>
+template <typename TA, bool GROUPED>
 static void launch_pan_warp(int vpl, dim3 grid, cudaStream_t stream, float* x, const void* delta, const float* post_w,
                             int post_kind, float post_eps, const float* w, int kind, float eps, void* out, const int* rows,
-                            int R, int H) {
+                            int R, int H, int post_groups, int groups) {
 #define PAN_WARP(V)                                                                                                       \
-    pico_launch((post_add_norm_warp_kernel<TA, V>), grid, dim3(128), 0, stream, x, (const TA*)delta, post_w, post_kind,    \
-                post_eps, w, kind, eps, (TA*)out, rows, R, H)
+    pico_launch((post_add_norm_warp_kernel<TA, V, GROUPED>), grid, dim3(128), 0, stream, x, (const TA*)delta, post_w, post_kind,    \
+                post_eps, w, kind, eps, (TA*)out, rows, R, H, post_groups, groups)
     if (vpl <= 1) PAN_WARP(1);
     else if (vpl <= 2) PAN_WARP(2);
     else if (vpl <= 4) PAN_WARP(4);
@@ -230,20 +288,31 @@ static void launch_pan_warp(int vpl, dim3 grid, cudaStream_t stream, float* x, c
 #undef PAN_WARP
 }
 
-// x float32 [*, H]; delta [*, H] or nullptr; out [R, H] or nullptr; rows int32 [R] or nullptr.
+// x float32 [*, H]; delta [*, H] or nullptr; out [R, H] or nullptr; rows int32 [R] or nullptr.  post_groups / groups: equal
+// runs an RMS norm of that side divides by a root mean square each (1: one for the row).
 PICO_API int pico_post_add_norm(float* x, const void* delta, const float* post_w, int post_kind, float post_eps,
                                 const float* w, int kind, float eps, void* out, const int* rows, int R, int H,
-                                int act_dtype, cudaStream_t stream) {
+                                int act_dtype, int post_groups, int groups, cudaStream_t stream) {
     if (R <= 0) return 0;
+    if (post_groups < 1 || groups < 1 || H % post_groups || H % groups || (post_groups > 1 && post_kind == NORM_CENTRED) ||
+        (groups > 1 && kind == NORM_CENTRED))
+        return PICO_ERR_SIZE;
+    const bool grouped = post_groups > 1 || groups > 1;
+    const bool v4 = H % 4 == 0 && (H / post_groups) % 4 == 0 && (H / groups) % 4 == 0;      // a vector lies within one group
     if (post_kind < 0 || post_kind > 2 || kind < 0 || kind > 3) return PICO_ERR_SIZE;
     if (act_dtype != PICO_F32 && act_dtype != PICO_BF16) return PICO_ERR_DTYPE;
-    if (H % 4 == 0 && H <= 2048) {       // a warp per row, the row in registers
+    if (v4 && H <= 2048) {       // a warp per row, the row in registers
         const int vpl = (H / 4 + 31) / 32;
         const dim3 grid((R + 3) / 4);
-        if (act_dtype == PICO_F32)
-            launch_pan_warp<float>(vpl, grid, stream, x, delta, post_w, post_kind, post_eps, w, kind, eps, out, rows, R, H);
-        else
-            launch_pan_warp<bf16>(vpl, grid, stream, x, delta, post_w, post_kind, post_eps, w, kind, eps, out, rows, R, H);
+#define PAN_ROWS(TA, GR)                                                                                                  \
+    launch_pan_warp<TA, GR>(vpl, grid, stream, x, delta, post_w, post_kind, post_eps, w, kind, eps, out, rows, R, H,       \
+                            post_groups, groups)
+        if (act_dtype == PICO_F32) {
+            if (grouped) PAN_ROWS(float, true); else PAN_ROWS(float, false);
+        } else {
+            if (grouped) PAN_ROWS(bf16, true); else PAN_ROWS(bf16, false);
+        }
+#undef PAN_ROWS
         return pico_launch_status();
     }
     const size_t smem = (size_t)(((H + 3) & ~3) + 33) * sizeof(float);
@@ -257,9 +326,8 @@ PICO_API int pico_post_add_norm(float* x, const void* delta, const float* post_w
         if (smem > 48 * 1024)                                                                                             \
             cudaFuncSetAttribute(post_add_norm_kernel<TA, V4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
         pico_launch((post_add_norm_kernel<TA, V4>), dim3(R), dim3(threads), smem, stream, x, (const TA*)delta, post_w,    \
-                    post_kind, post_eps, w, kind, eps, (TA*)out, rows, H);                                                \
+                    post_kind, post_eps, w, kind, eps, (TA*)out, rows, H, post_groups, groups);                           \
     } while (0)
-    const bool v4 = H % 4 == 0;
     if (act_dtype == PICO_F32) {
         if (v4) LAUNCH_PAN(float, true); else LAUNCH_PAN(float, false);
     } else if (act_dtype == PICO_BF16) {

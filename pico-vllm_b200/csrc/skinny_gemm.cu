@@ -14,6 +14,7 @@
 //   STORE     y = (sum + bias) as bfloat16 or float32                       (plain projection, head)
 //   RESIDUAL  x_res[m, n] += sum, float32 in place                          (o_proj, down_proj)
 //   SWIGLU    a[m, i] = silu(gate_i) * up_i; rows i (gate) and I + i (up)   (gate_up, no 2I buffer)
+//   CAPPED    the same rows, a[m, i] = g sigmoid(1.702 g) (u + 1) with g = min(gate_i, L), u = clamp(up_i, -L, L)
 //   ROPE      q/k heads: rows d and d + hd/2 of a head: bias, rotation by the token's position,
 //             q to the query buffer, k and v straight into their cache pages   (qkv projection)
 //   ARGMAX    token[m] = the first n with the largest sum: every block keeps the best of its own tiles, the
@@ -50,7 +51,8 @@
 #define SG_CTAS_PER_SM 2
 #endif
 
-enum { SG_STORE = 0, SG_RESIDUAL = 1, SG_SWIGLU = 2, SG_ROPE = 3, SG_ARGMAX = 4 };
+enum { SG_STORE = 0, SG_RESIDUAL = 1, SG_SWIGLU = 2, SG_ROPE = 3, SG_ARGMAX = 4, SG_CAPPED = 5 };
+__host__ __device__ constexpr bool sg_is_glu(int epi) { return epi == SG_SWIGLU || epi == SG_CAPPED; }
 
 // ARGMAX: what each block found, and how many blocks have reported (reset by the block that reports last, so
 // launches on one stream need no clearing in between; launches that overlap on the GPU would mix their entries)
@@ -77,7 +79,8 @@ struct SkinnyArgs {
     const float* bias;        // [N] or null (STORE and ROPE)
     // RESIDUAL
     float* resid;             // [M, N]
-    // SWIGLU: N = 2 * I; out = [M, I] bf16 in `out`
+    // SWIGLU, CAPPED: N = 2 * I; out = [M, I] bf16 in `out`
+    float limit;              // CAPPED: L of g' sigmoid(1.702 g') (u' + 1), g' = min(g, L), u' = clamp(u, -L, L)
     // ROPE
     int nh, nkv, hd, rot_half, page_size;
     const int* positions;     // [M]
@@ -113,7 +116,7 @@ __device__ __forceinline__ void sg_mma(float (&d)[4], const uint32_t (&a)[4], ui
 // The two runs of 8 weight rows a block owns.
 template <int EPI>
 __device__ __forceinline__ void sg_rows(const SkinnyArgs& p, int tile, int& row_a, int& row_b) {
-    if (EPI == SG_SWIGLU) {
+    if (sg_is_glu(EPI)) {
         row_a = tile * 8;                  // gate rows
         row_b = p.N / 2 + tile * 8;        // the same features' up rows
     } else if (EPI == SG_ROPE) {
@@ -174,15 +177,21 @@ __device__ __forceinline__ void sg_epilogue(const SkinnyArgs& p, const float* re
                 else reinterpret_cast<bf16*>(p.out)[(size_t)t * p.ld_out + n] = __float2bfloat16_rn(y);
             }
         }
-    } else if (EPI == SG_SWIGLU) {
+    } else if (sg_is_glu(EPI)) {
         for (int idx = threadIdx.x; idx < 8 * XR; idx += SG_THREADS) {
             const int t = idx / 8, f = idx - t * 8;
             if (t >= p.M) continue;
             const float gte = sg_sum<XR>(red, f, t);
             const int fu = f + 8;
             const float up = sg_sum<XR>(red, fu, t);
-            const float sl = gte / (1.0f + expf(-gte));
-            reinterpret_cast<bf16*>(p.out)[(size_t)t * p.ld_out + row_a + f] = __float2bfloat16_rn(sl * up);
+            float y;
+            if (EPI == SG_CAPPED) {
+                const float gc = fminf(gte, p.limit), uc = fminf(fmaxf(up, -p.limit), p.limit);
+                y = gc / (1.0f + expf(-1.702f * gc)) * (uc + 1.0f);
+            } else {
+                y = gte / (1.0f + expf(-gte)) * up;
+            }
+            reinterpret_cast<bf16*>(p.out)[(size_t)t * p.ld_out + row_a + f] = __float2bfloat16_rn(y);
         }
     } else {    // SG_ROPE
         const int rot_heads = p.nh + p.nkv;
@@ -557,14 +566,15 @@ PICO_API int pico_skinny_linear_residual(const void* x, int ldx, const void* w, 
     return sg_launch<SG_RESIDUAL>(a, N / 16, stream);
 }
 
-// out[M, I] = silu(x wg^T) * (x wu^T) with w = [wg; wu] of shape [2I, K].  I % 8 == 0.
+// out[M, I] = silu(x wg^T) * (x wu^T) with w = [wg; wu] of shape [2I, K], or with limit > 0 the capped form of the two
+// products (see SkinnyArgs).  I % 8 == 0.
 PICO_API int pico_skinny_gate_up_swiglu(const void* x, int ldx, const void* w, void* out, int M, int I, int K,
-                                        const float* norm_w, float eps, cudaStream_t stream) {
+                                        const float* norm_w, float eps, float limit, cudaStream_t stream) {
     if (sg_check(M, 2 * I, K, norm_w ? 8 : ldx) || I % 8 != 0) return PICO_ERR_SIZE;
     SkinnyArgs a = {};
     a.w = (const bf16*)w; sg_set_x(a, x, ldx, norm_w, eps, nullptr); a.M = M; a.N = 2 * I; a.K = K;
-    a.out = out; a.ld_out = I;
-    return sg_launch<SG_SWIGLU>(a, I / 8, stream);
+    a.out = out; a.ld_out = I; a.limit = limit;
+    return limit > 0.f ? sg_launch<SG_CAPPED>(a, I / 8, stream) : sg_launch<SG_SWIGLU>(a, I / 8, stream);
 }
 
 // qkv projection with bias, rotary encoding and cache store fused: q_out [M, nh*hd] gets the rotated

@@ -50,6 +50,9 @@ class Batch:
     # int32, one entry per wanted row: when given, the head may write the greedy token of every wanted row here and
     # return no logits
     greedy_out: Optional[torch.Tensor] = None
+    # what one part of the model hands to later ones within a step (an early layer's values, for instance), by a name the
+    # parts agree on; rows are the batch's tokens.  Emptied when a forward pass starts.
+    carry: Dict[str, torch.Tensor] = field(default_factory=dict)
 
     def plan(self, mixer):
         """The plan ``mixer.plan(shape)`` returned for this step, or None."""

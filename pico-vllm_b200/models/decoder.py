@@ -107,6 +107,7 @@ class DecoderModel:
         """Runs the batch's tokens through every call of the order; returns float32 logits
         [len(batch.logit_rows), vocab] - or None when ``batch.greedy_out`` was given and the head wrote the
         greedy token of every wanted row there instead."""
+        batch.carry.clear()
         x = self.embed.forward(batch.token_ids, batch.feedback)
         if self.embed_position is not None:
             x = self.embed_position.add_to(x, batch.positions)

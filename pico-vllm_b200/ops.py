@@ -53,32 +53,35 @@ def library():
         "pico_swiglu": [vp, vp, i32, i32, i32, vp],
         "pico_rope_store": [vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp],
         "pico_paged_attention_generic": [vp, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32,
-                                         i32, i32, f32, i32, f32, i32, vp, i32, vp, vp],
+                                         i32, i32, f32, i32, f32, i32, vp, i32, vp, vp, vp],
         "pico_paged_prefill_mma": [vp, i32, vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, f32, vp, i32,
-                                   vp, vp],
+                                   vp, vp, vp],
         "pico_paged_decode_mma": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32,
-                                  f32, i32, f32, vp, i32, vp, vp],
+                                  f32, i32, f32, vp, i32, vp, vp, vp],
         "pico_skinny_linear": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp, f32, vp, vp],
         "pico_skinny_argmax": [vp, i32, vp, vp, i32, i32, i32, vp, f32, vp, vp],
         "pico_skinny_norm_fits": [i32, i32],
         "pico_skinny_linear_residual": [vp, i32, vp, vp, i32, i32, i32, vp],
-        "pico_skinny_gate_up_swiglu": [vp, i32, vp, vp, i32, i32, i32, vp, f32, vp],
+        "pico_skinny_gate_up_swiglu": [vp, i32, vp, vp, i32, i32, i32, vp, f32, f32, vp],
         "pico_skinny_qkv_rope_store": [vp, i32, vp, vp, vp, vp, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, f32,
                                        vp],
         "pico_make_kv_tensor_map": [vp, vp, i64, i32, i32],
         "pico_paged_decode_tma": [vp, vp, vp, i32, vp, vp, vp, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32,
-                                  f32, i32, i32, f32, vp],
+                                  f32, i32, i32, f32, vp, vp, vp, vp],
         "pico_tma_status": [vp],
         "pico_make_kv_tensor_map_2d": [vp, vp, i64, i32, i32, i32],
         "pico_paged_prefill_tcgen05": [vp, vp, vp, i32, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32,
-                                       vp, i32, vp, i32, f32, vp, i32, vp, vp],
+                                       vp, i32, vp, i32, f32, vp, i32, vp, vp, vp],
         "pico_tca_status": [vp],
-        "pico_gemm_tcgen05_pair": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp],
+        "pico_gemm_tcgen05_pair": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp],
         "pico_tp_status": [vp],
         "pico_sample": [vp, i32, i32, i32, vp, vp, vp, vp, vp],
-        "pico_post_add_norm": [vp, vp, vp, i32, f32, vp, i32, f32, vp, vp, i32, i32, i32, vp],
+        "pico_post_add_norm": [vp, vp, vp, i32, f32, vp, i32, f32, vp, vp, i32, i32, i32, i32, i32, vp],
         "pico_scale_softcap": [vp, i32, i32, i32, f32, f32, vp],
-        "pico_latent_norm_store": [vp, i32, i32, i32, vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32, i32, i32, vp],
+        "pico_latent_norm_store": [vp, i32, i32, i32, vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32, i32, i32, i32, i32, i32, vp, f32,
+                                   vp, vp],
+        "pico_rotate_tail": [vp, i32, i32, i32, i32, i32, i32, vp, f32, vp, i32, vp],
+        "pico_head_norm_store": [vp, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp],
         "pico_head_scale": [vp, vp, i32, i32, i32, i32, vp],
         "pico_moe_route": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, i32, vp, f32, i32, i32, i32, vp],
         "pico_moe_group": [vp, i32, i32, i32, vp, vp, vp, vp, vp],
@@ -264,10 +267,11 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
                     n_heads: int, n_kv_heads: int, head_dim: int, page_size: int, window: Optional[int],
                     scale: float, n_splits: int = 1, scratch: Optional[torch.Tensor] = None,
                     softcap: Optional[float] = None, slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, rates: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of every token of the batch over its request's cache pages.
     ``softcap`` c: the scaled score s becomes c * tanh(s / c) before the softmax.
-    ``slopes`` float32 [n_heads]: slopes[h] * (query position - key position) is taken off head h's scores.
+    ``slopes`` float32 [n_heads]: slopes[h] * (query position - key position) is taken off head h's scores; with ``rates``
+    float32 [n_heads] it is slopes[h] * ln(1 + rates[h] * (query position - key position)).
     ``chunk`` C: the token at position p sees only keys from floor(p / C) * C on (positions count from the request's start).
     ``sinks`` float32 [n_heads]: head h's softmax has one more term exp(sinks[h]) in its denominator and no value for it.
 
@@ -279,8 +283,8 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
     """
     _cuda(q, k_pages, v_pages, out, tok_seg, positions, block_table, scratch)
     T = q.shape[0]
-    if head_dim % 16 != 0 or head_dim > 256:
-        raise KernelError(f"paged_attention: head_dim must be a multiple of 16 up to 256, got {head_dim}")
+    if head_dim % 16 != 0 or head_dim > 640:
+        raise KernelError(f"paged_attention: head_dim must be a multiple of 16 up to 640, got {head_dim}")
     if n_heads % n_kv_heads != 0:
         raise KernelError("paged_attention: n_heads must be a multiple of n_kv_heads")
     if q.stride(1) != 1 or q.shape[1] < n_heads * head_dim or out.shape != (T, n_heads * head_dim):
@@ -294,10 +298,7 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
     for t in (tok_seg, positions, block_table):
         if t.dtype != torch.int32:
             raise KernelError("paged_attention: index tensors must be int32")
-    _cuda(slopes, sinks)
-    for t in (slopes, sinks):
-        if t is not None and (t.dtype != torch.float32 or t.shape != (n_heads,)):
-            raise KernelError("paged_attention: slopes and sinks must be float32 [n_heads]")
+    _check_bias(slopes, sinks, rates, n_heads, "paged_attention")
     part_o = part_ml = None
     if n_splits > 1:
         need = attention_scratch_floats(T, n_heads, head_dim, n_splits)
@@ -309,10 +310,19 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), part_o, part_ml, _ptr(tok_seg),
         _ptr(positions), _ptr(block_table), block_table.stride(0), T, n_heads, n_kv_heads, head_dim, page_size,
         int(window) if window else 0, float(scale), n_splits, float(softcap) if softcap else 0.0, _dtype_code(q),
-        _ptr(slopes), int(chunk) if chunk else 0, _ptr(sinks), _stream()),
+        _ptr(slopes), int(chunk) if chunk else 0, _ptr(sinks), _ptr(rates), _stream()),
         f"paged_attention (head_dim {head_dim})")
     _count(2 if n_splits > 1 else 1)
     return out
+
+
+def _check_bias(slopes, sinks, rates, n_heads: int, what: str) -> None:
+    _cuda(slopes, sinks, rates)
+    for t in (slopes, sinks, rates):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (n_heads,) or not t.is_contiguous()):
+            raise KernelError(f"{what}: slopes, sinks and rates must be float32 [n_heads]")
+    if rates is not None and slopes is None:
+        raise KernelError(f"{what}: rates of a distance bias need its slopes")
 
 
 def mma_attention_takes(dtype: torch.dtype, n_heads: int, n_kv_heads: int, head_dim: int) -> bool:
@@ -405,7 +415,8 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
                         scale: float, n_splits: int = 1, scratch: Optional[torch.Tensor] = None,
                         k_map=None, v_map=None, k_map2d=None, v_map2d=None, pair_min_keys: int = 0,
                         softcap: Optional[float] = None, slopes: Optional[torch.Tensor] = None,
-                        chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
+                        rates: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The same attention as :func:`paged_attention` for bfloat16 on tensor cores, in two launches:
     segments that bring two or more tokens (``prefill_segs`` int32 [n_prefill_segs], None = all
     segments; ``cu_q`` int32 [segments + 1]; ``max_prefill_q`` their longest) and single tokens
@@ -414,8 +425,8 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     With ``k_map`` / ``v_map`` (from :func:`make_kv_tensor_map` over these same pages) the single
     tokens run in the kernel that brings pages in by TMA; with ``k_map2d`` / ``v_map2d`` (from
     :func:`make_kv_tensor_map_2d`) the portions run on the tcgen05 tensor cores.
-    ``slopes``, ``chunk`` and ``sinks`` as in :func:`paged_attention` (not together with ``softcap``); with them the
-    single tokens run in the kernel that reads pages through the block table."""
+    ``slopes``, ``chunk``, ``sinks`` and ``rates`` as in :func:`paged_attention` (not together with ``softcap``); with
+    ``chunk`` the single tokens run in the kernel that reads pages through the block table."""
     _cuda(q, k_pages, v_pages, out, tok_seg, positions, block_table, cu_q, prefill_segs, decode_tokens, scratch)
     T = q.shape[0]
     if not mma_attention_takes(q.dtype, n_heads, n_kv_heads, head_dim):
@@ -432,10 +443,7 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     for t in (tok_seg, positions, block_table, cu_q, prefill_segs, decode_tokens):
         if t is not None and t.dtype != torch.int32:
             raise KernelError("paged_attention_mma: index tensors must be int32")
-    _cuda(slopes, sinks)
-    for t in (slopes, sinks):
-        if t is not None and (t.dtype != torch.float32 or t.shape != (n_heads,)):
-            raise KernelError("paged_attention_mma: slopes and sinks must be float32 [n_heads]")
+    _check_bias(slopes, sinks, rates, n_heads, "paged_attention_mma")
     lib = library()
     win = int(window) if window else 0
     cap = float(softcap) if softcap else 0.0
@@ -443,7 +451,7 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     extra = slopes is not None or sinks is not None or chunk > 0
     if extra and cap > 0.0:
         raise KernelError("paged_attention_mma: a distance bias, chunks or a sink are not built together with a soft cap")
-    if extra:
+    if chunk > 0:
         k_map = v_map = None
     if n_prefill_segs > 0 and k_map2d is not None and v_map2d is not None:
         # pair_min_keys > 0 (and scratch for two partial results per (token, head)): every query tile gets two
@@ -458,7 +466,7 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
                                               n_kv_heads, head_dim, page_size, win, float(scale),
                                               int(pair_min_keys) if split else 0, _ptr(scratch) if split else None, T,
                                               _ptr(counters) if split else None, counters.numel() if split else 0,
-                                              cap, _ptr(slopes), chunk, _ptr(sinks), _stream()),
+                                              cap, _ptr(slopes), chunk, _ptr(sinks), _ptr(rates), _stream()),
                f"paged_prefill_tcgen05 (head_dim {head_dim})")
         _count()
     elif n_prefill_segs > 0:
@@ -466,7 +474,7 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
                                           _ptr(prefill_segs), n_prefill_segs, _ptr(cu_q), max_prefill_q,
                                           _ptr(positions), _ptr(block_table), block_table.stride(0), n_heads,
                                           n_kv_heads, head_dim, page_size, win, float(scale), cap, _ptr(slopes), chunk,
-                                          _ptr(sinks), _stream()),
+                                          _ptr(sinks), _ptr(rates), _stream()),
                f"paged_prefill_mma (head_dim {head_dim})")
         _count()
     if n_decode_tokens > 0:
@@ -482,14 +490,15 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
                                              _ptr(decode_tokens), n_decode_tokens, _ptr(tok_seg), _ptr(positions),
                                              _ptr(block_table), block_table.stride(0), n_heads, n_kv_heads,
                                              head_dim, page_size, win, float(scale), n_splits,
-                                             1 if k_pages.data_ptr() == v_pages.data_ptr() else 0, cap, _stream()),
+                                             1 if k_pages.data_ptr() == v_pages.data_ptr() else 0, cap,
+                                             _ptr(slopes), _ptr(sinks), _ptr(rates), _stream()),
                    f"paged_decode_tma (head_dim {head_dim})")
         else:
             _check(lib.pico_paged_decode_mma(_ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), part_o,
                                              part_ml, _ptr(decode_tokens), n_decode_tokens, _ptr(tok_seg),
                                              _ptr(positions), _ptr(block_table), block_table.stride(0), n_heads,
                                              n_kv_heads, head_dim, page_size, win, float(scale), n_splits, cap,
-                                             _ptr(slopes), chunk, _ptr(sinks), _stream()),
+                                             _ptr(slopes), chunk, _ptr(sinks), _ptr(rates), _stream()),
                    f"paged_decode_mma (head_dim {head_dim})")
         clustered = k_map is not None and v_map is not None and n_splits in (2, 4, 8, 16)
         _count(2 if n_splits > 1 and not clustered else 1)
@@ -591,8 +600,9 @@ def skinny_linear_residual(x: torch.Tensor, weight: torch.Tensor, residual: torc
 
 
 def skinny_gate_up_swiglu(x: torch.Tensor, gate_up_weight: torch.Tensor, norm_weight: Optional[torch.Tensor] = None,
-                          eps: float = 0.0) -> torch.Tensor:
-    """silu(x wg^T) * (x wu^T) for gate_up_weight = [wg; wu] ([2I, K]); returns [M, I] bfloat16.
+                          eps: float = 0.0, limit: Optional[float] = None) -> torch.Tensor:
+    """silu(x wg^T) * (x wu^T) for gate_up_weight = [wg; wu] ([2I, K]); returns [M, I] bfloat16.  With ``limit`` L the capped
+    form instead: g sigmoid(1.702 g) (u + 1) with g = min(x wg^T, L) and u = clamp(x wu^T, -L, L).
     With ``norm_weight``: x is the float32 residual stream and is RMS-normed on the way in."""
     _cuda(x, gate_up_weight, norm_weight)
     if _norm_args(x, norm_weight, "skinny_gate_up_swiglu") is not None:
@@ -604,7 +614,7 @@ def skinny_gate_up_swiglu(x: torch.Tensor, gate_up_weight: torch.Tensor, norm_we
     I = gate_up_weight.shape[0] // 2
     out = torch.empty((M, I), dtype=torch.bfloat16, device=x.device)
     _check(library().pico_skinny_gate_up_swiglu(_ptr(x), x.stride(0), _ptr(gate_up_weight), _ptr(out), M, I, K,
-                                                _ptr(norm_weight), float(eps), _stream()), "skinny_gate_up_swiglu")
+                                                _ptr(norm_weight), float(eps), float(limit or 0.0), _stream()), "skinny_gate_up_swiglu")
     _count()
     return out
 
@@ -670,11 +680,11 @@ def tc_status() -> int:
 TC_PAIR_MIN_TOKENS = 200      # from here on the tcgen05 path pays
 
 
-def _tc_gemm(x, weight, out, residual, M, N, K, epi, rows, what):
+def _tc_gemm(x, weight, out, residual, M, N, K, epi, rows, what, limit=0.0):
     """The tcgen05 product kernel: a tile per pair of blocks (``tcgen05.mma.cta_group::2``).  ``rows``: None = the
     kernel picks its tile; 256 or 512 = that many rows of x per pair."""
     _check(library().pico_gemm_tcgen05_pair(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), _ptr(residual), M, N, K,
-                                            epi, int(rows or 0), _stream()), "gemm_tcgen05_pair" + what)
+                                            epi, int(rows or 0), float(limit), _stream()), "gemm_tcgen05_pair" + what)
     _count()
 
 
@@ -701,15 +711,16 @@ def tc_linear_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.Te
     _tc_gemm(x, weight, None, residual, M, N, K, 1, rows, " (residual)")
 
 
-def tc_gate_up_swiglu(x: torch.Tensor, gate_up_weight: torch.Tensor, rows=None) -> torch.Tensor:
-    """silu(x wg^T) * (x wu^T) for gate_up_weight = [wg; wu]; returns [M, I] bfloat16."""
+def tc_gate_up_swiglu(x: torch.Tensor, gate_up_weight: torch.Tensor, rows=None, limit: Optional[float] = None) -> torch.Tensor:
+    """silu(x wg^T) * (x wu^T) for gate_up_weight = [wg; wu]; returns [M, I] bfloat16.  ``limit``: the capped form, as in
+    :func:`skinny_gate_up_swiglu`."""
     _cuda(x, gate_up_weight)
     if not tc_takes(x, gate_up_weight):
         raise KernelError("tc_gate_up_swiglu: sizes not taken")
     M, K = x.shape
     I = gate_up_weight.shape[0] // 2
     out = torch.empty((M, I), dtype=torch.bfloat16, device=x.device)
-    _tc_gemm(x, gate_up_weight, out, None, M, 2 * I, K, 2, rows, " (swiglu)")
+    _tc_gemm(x, gate_up_weight, out, None, M, 2 * I, K, 3 if limit else 2, rows, " (gate_up)", limit or 0.0)
     return out
 
 
@@ -771,13 +782,14 @@ def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor], top_p: Opt
 # Norm of a sublayer's output, residual add and the next norm in one kernel.
 def post_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post_weight: Optional[torch.Tensor], post_kind: int,
                   post_eps: float, weight: Optional[torch.Tensor], kind: int, eps: float, out: Optional[torch.Tensor],
-                  rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                  rows: Optional[torch.Tensor] = None, post_groups: int = 1, groups: int = 1) -> Optional[torch.Tensor]:
     """x float32 [T, H] += N_post(delta) (written back unless ``rows`` picks rows), out = N(x).
 
     ``post_kind`` / ``kind``: NORM_NONE, NORM_RMS (u / sqrt(mean u^2 + eps) * w) or NORM_CENTRED ((u - mean u) /
     sqrt(mean (u - mean u)^2 + eps) * w); weights float32 [H].  delta (or None) and out are in the activation
     type; with ``rows`` (int32 [R]) out[r] is computed from row rows[r] and x is left alone; ``out`` None: the add
-    alone."""
+    alone.  ``post_groups`` / ``groups``: that RMS norm divides each of so many equal runs of the row by the run's own
+    root mean square."""
     _cuda(x, delta, post_weight, weight, out, rows)
     H = x.shape[1]
     R = rows.shape[0] if rows is not None else x.shape[0]
@@ -788,6 +800,9 @@ def post_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post_weight: O
             raise KernelError(f"post_add_norm: unknown kind of norm {k}")
         if w is not None and (w.dtype != torch.float32 or w.shape != (H,)):
             raise KernelError(f"post_add_norm: {what} must be float32 [H]")
+    for n, k in ((post_groups, post_kind), (groups, kind)):
+        if n < 1 or H % n or (n > 1 and k == NORM_CENTRED):
+            raise KernelError(f"post_add_norm: a row of {H} in {n} groups (equal groups, RMS norms only)")
     if out is None and delta is None:
         return None
     like = out if out is not None else delta
@@ -799,7 +814,8 @@ def post_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post_weight: O
         raise KernelError("post_add_norm: rows must be int32")
     _check(library().pico_post_add_norm(_ptr(x), _ptr(delta), _ptr(post_weight), int(post_kind), float(post_eps),
                                         _ptr(weight), int(kind) if out is not None else NORM_NONE, float(eps), _ptr(out),
-                                        _ptr(rows), R, H, _dtype_code(like), _stream()), f"post_add_norm (width {H})")
+                                        _ptr(rows), R, H, _dtype_code(like), int(post_groups), int(groups), _stream()),
+           f"post_add_norm (width {H})")
     _count()
     return out
 
@@ -819,15 +835,21 @@ def scale_softcap(logits: torch.Tensor, scale: float, cap: Optional[float]) -> t
 # Latent attention: what stands between its matrix products.
 def latent_norm_store(proj: torch.Tensor, q_off: int, q_rank: int, q_weight: Optional[torch.Tensor], kv_off: int, kv_rank: int,
                       kv_weight: Optional[torch.Tensor], slots: Optional[torch.Tensor], cache: Optional[torch.Tensor],
-                      g_off: int, heads: int, eps: float):
+                      g_off: int, heads: int, eps: float, rot=None):
     """From a token's down projection row ``proj[t]`` (query latent at q_off, key/value latent at kv_off, one gate
     logit per head at g_off): the RMS-normed query latent [T, q_rank], the RMS-normed key/value latent into cache
     row ``slots[t]`` (``cache`` [..., row width >= kv_rank], zero beyond kv_rank; nothing for a slot of -1;
     kv_rank 0: no key/value part), and sigmoid of the gate logits (float32 [T, heads]).  ``q_rank`` 0: no query latent,
-    ``heads`` 0: no gate; the part that is absent comes back as None.  Returns (cq, gate)."""
+    ``heads`` 0: no gate; the part that is absent comes back as None.  ``rot`` (offset, dim, positions, inv_freq, mult): the
+    row also holds a key part of ``dim`` numbers shared by all heads; its dims i and i + n/2 (n = 2 len(inv_freq) <= dim) turn
+    by position * inv_freq[i], cos and sin times ``mult``, and it is stored behind the latent.  Returns (cq, gate)."""
     _cuda(proj, q_weight, kv_weight, slots, cache)
     T = proj.shape[0]
-    if proj.stride(1) != 1 or max(q_off + q_rank, kv_off + kv_rank, g_off + heads) > proj.shape[1]:
+    r_off, r_dim, r_pos, r_freq, r_mult = rot if rot is not None else (0, 0, None, None, 1.0)
+    _cuda(r_pos, r_freq)
+    if r_dim > 0 and (r_pos.dtype != torch.int32 or r_freq.dtype != torch.float32 or 2 * r_freq.shape[0] > r_dim):
+        raise KernelError("latent_norm_store: rotation needs int32 positions and at most dim / 2 float32 frequencies")
+    if proj.stride(1) != 1 or max(q_off + q_rank, kv_off + kv_rank, g_off + heads, r_off + r_dim) > proj.shape[1]:
         raise KernelError("latent_norm_store: the projection row is narrower than its parts")
     if q_rank > 0 and (q_weight is None or q_weight.dtype != torch.float32 or q_weight.shape != (q_rank,)):
         raise KernelError("latent_norm_store: q_weight must be float32 [q_rank]")
@@ -836,17 +858,66 @@ def latent_norm_store(proj: torch.Tensor, q_off: int, q_rank: int, q_weight: Opt
         if kv_weight is None or kv_weight.dtype != torch.float32 or kv_weight.shape != (kv_rank,):
             raise KernelError("latent_norm_store: kv_weight must be float32 [kv_rank]")
         if slots is None or slots.dtype != torch.int32 or slots.shape[0] != T or cache is None \
-                or cache.dtype != proj.dtype or not cache.is_contiguous() or cache.shape[-1] < kv_rank:
+                or cache.dtype != proj.dtype or not cache.is_contiguous() or cache.shape[-1] < kv_rank + r_dim:
             raise KernelError("latent_norm_store: needs int32 slots and a contiguous cache of the activation type")
         row = cache.shape[-1]
     cq = torch.empty((T, q_rank), dtype=proj.dtype, device=proj.device) if q_rank > 0 else None
     gate = torch.empty((T, heads), dtype=torch.float32, device=proj.device) if heads > 0 else None
     _check(library().pico_latent_norm_store(_ptr(proj), proj.stride(0), q_off, q_rank, _ptr(q_weight), _ptr(cq), kv_off,
                                             kv_rank, _ptr(kv_weight), _ptr(slots), _ptr(cache) if kv_rank > 0 else None,
-                                            row, g_off, heads, _ptr(gate), float(eps), T, _dtype_code(proj), _stream()),
+                                            row, g_off, heads, _ptr(gate), float(eps), T, _dtype_code(proj), r_off, r_dim,
+                                            2 * r_freq.shape[0] if r_dim > 0 else 0, _ptr(r_freq), float(r_mult), _ptr(r_pos),
+                                            _stream()),
            "latent_norm_store")
     _count()
     return cq, gate
+
+
+def rotate_tail(x: torch.Tensor, heads: int, rot_dim: int, positions: torch.Tensor, inv_freq: torch.Tensor,
+                mult: float = 1.0) -> torch.Tensor:
+    """In place on x [T, heads * w]: of the last ``rot_dim`` numbers of every head, dims i and i + n/2 (n = 2 len(inv_freq))
+    turn by position * inv_freq[i], cos and sin times ``mult``; the rest stays.  Rows of position -1 are left alone."""
+    _cuda(x, positions, inv_freq)
+    T = x.shape[0]
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] % heads or positions.dtype != torch.int32 or positions.shape != (T,) \
+            or inv_freq.dtype != torch.float32 or 2 * inv_freq.shape[0] > rot_dim:
+        raise KernelError("rotate_tail: x [T, heads * w], int32 positions [T], at most rot_dim / 2 float32 frequencies")
+    _check(library().pico_rotate_tail(_ptr(x), x.stride(0), T, heads, x.shape[1] // heads, rot_dim, 2 * inv_freq.shape[0],
+                                      _ptr(inv_freq), float(mult), _ptr(positions), _dtype_code(x), _stream()), "rotate_tail")
+    _count()
+    return x
+
+
+def head_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, norm: bool, eps: float, slots: Optional[torch.Tensor],
+                    k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int,
+                    vdim: int, row: int, page_size: int, mix: Optional[torch.Tensor] = None,
+                    first: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per token row [q heads | k heads | v heads]: with ``norm`` every query and key head divided by its own root mean square
+    (no weight); with ``mix`` (one float32 number on the device) and ``first`` [T, kv_heads * vdim] the values become
+    (1 - mix) v + mix first.  Keys and values go to their cache rows, heads padded with zeros to ``row``; returns the queries
+    [T, heads * row] in proj's type."""
+    _cuda(proj, slots, k_pages, v_pages, mix, first)
+    T = proj.shape[0]
+    if proj.stride(1) != 1 or max(q_off + heads * dim, k_off + kv_heads * dim, v_off + kv_heads * vdim) > proj.shape[1] or row < max(dim, vdim):
+        raise KernelError("head_norm_store: the projection row is narrower than its parts, or a head wider than its row")
+    if slots is not None:
+        if slots.dtype != torch.int32 or k_pages is None or v_pages is None:
+            raise KernelError("head_norm_store: slots must be int32 and come with pages")
+        for pg in (k_pages, v_pages):
+            if pg.dtype != proj.dtype or not pg.is_contiguous() or tuple(pg.shape[1:]) != (kv_heads, page_size, row):
+                raise KernelError("head_norm_store: pages must be contiguous [pages, kv_heads, page_size, row] in proj's type")
+    if (mix is None) != (first is None):
+        raise KernelError("head_norm_store: mixed values need both the number and the other values")
+    if mix is not None and (mix.dtype != torch.float32 or mix.numel() != 1 or first.dtype != proj.dtype or first.stride(1) != 1
+                            or first.shape != (T, kv_heads * vdim)):
+        raise KernelError("head_norm_store: mix is one float32 number and first [T, kv_heads * vdim] in proj's type")
+    q = torch.empty((T, heads * row), dtype=proj.dtype, device=proj.device)
+    _check(library().pico_head_norm_store(_ptr(proj), proj.stride(0), q_off, k_off, v_off, 1 if norm else 0, float(eps), _ptr(slots),
+                                          _ptr(k_pages), _ptr(v_pages), _ptr(q), _ptr(mix), _ptr(first),
+                                          first.stride(0) if first is not None else 0, T, heads, kv_heads, dim, vdim, row, page_size,
+                                          _dtype_code(proj), _stream()), "head_norm_store")
+    _count()
+    return q
 
 
 def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -1,6 +1,6 @@
 from .base import Param, Piece, Part, PagedKV, PagedTensors, PagedLatent, FixedState, CacheView, StepShape, MixerPlan
 from .registry import register, make, MIXERS, FEED_FORWARDS, NORMS, POSITIONS
-from .norm import RMSNorm, CentredNorm, NormedDelta, PassNorm, ScalarRMSNorm
+from .norm import RMSNorm, CentredNorm, NormedDelta, PassNorm, ScalarRMSNorm, GroupedRMSNorm
 from .rotary import Rotary, NoPosition, YarnRotary
 from .attention import GQAAttention, QKNormAttention
 from .linear_attention import DecayLinearAttention
@@ -22,4 +22,4 @@ __all__ = ["Param", "Piece", "Part", "PagedKV", "PagedTensors", "FixedState", "C
            "LatentAttention", "RoutedExperts", "SandwichBlock", "PassNorm", "YarnRotary", "QKNormAttention",
            "DecayLinearAttention", "ScalarRMSNorm", "LearnedPositions", "HyperConnection", "HyperDelta", "HyperBlock",
            "ExpGatedMatrixMemory", "ForgetWriteLinearAttention", "StateSpaceDuality", "DistanceBiasAttention", "ParallelMixers",
-           "TokenSideTable", "TokenSideInput", "ConvRopeAttention", "GatedDeltaRule", "SumDelta", "ParallelBlock"]
+           "TokenSideTable", "TokenSideInput", "ConvRopeAttention", "GatedDeltaRule", "SumDelta", "ParallelBlock", "GroupedRMSNorm"]

@@ -27,14 +27,14 @@ class AttentionPlan(MixerPlan):
                                # that sees at least this many keys (two partial results per token and head in scratch)
 
 
-def decode_splits(shape: StepShape, n_kv_heads: int) -> int:
+def decode_splits(shape: StepShape, n_kv_heads: int, window: Optional[int] = None) -> int:
     """How many parts to cut each single token's key range into: a power of two (the parts of one
     token and kv head run as one thread-block cluster): up to 16 while that is at most one block
     per SM, else up to 8 while the blocks make no more than one wave of two per SM; each part at
-    least two tiles of 64 keys."""
+    least two tiles of 64 keys of the context, or of the ``window`` a token sees of it."""
     groups = max(1, shape.num_tokens * n_kv_heads)
     want = 16 if groups * 16 <= shape.num_sms else min(2 * shape.num_sms // groups, 8)
-    want = min(want, shape.max_kv // 128)
+    want = min(want, (shape.max_kv if window is None else min(shape.max_kv, window)) // 128)
     splits = 1
     while splits * 2 <= want:
         splits *= 2

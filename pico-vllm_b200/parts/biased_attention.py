@@ -8,6 +8,14 @@
     s(i, j) = scale * q_i . k_j - slope_h * (i - j),   slope_h = 2^(-8 (h + 1) / H)                     (distance_bias)
     chunk C:        position i sees j <= i only when floor(i / C) = floor(j / C), counted from the request's start
     sink:           p_j = exp(s_j) / (exp(sink) + sum_j exp(s_j)) with sink = 0: a key of score 0 that has no value
+    learned_sink:   the same with a learned number per head (tensor ``sink``)
+    head_qk_norm:   each head's q and k divided by its own root mean square (no weight), instead of whole_qk_norm
+    log_bias:       r1_h * ln(1 + r2_h * (i - j)) is taken off the score, r1 and r2 learned numbers per head (tensors ``r1``,
+                    ``r2``), instead of the fixed slopes
+    value_mix:      a group of layers shares the first one's values: "first" hands its projected values on under ``mix_key``
+                    for the rest of the step, "mix" reads them, v <- (1 - lambda) v + lambda v_first with the learned number
+                    lambda (tensor ``vmix``); what is cached is the mixed v.  (The first layer's lambda is loaded, not used.)
+    window W:       position i sees the last W positions, itself included
     out = W_o concat_heads(sum_j p_j v_j)
 
 Launches: one product for q, k, v -> norms and cache store (one kernel) -> paged attention -> output product.  Norms, scores
@@ -25,6 +33,7 @@ from typing import List, Optional
 import torch
 
 from .. import ops
+from ..errors import ConfigError
 from .attention import AttentionPlan, _linear, decode_splits
 from .base import CacheView, MixerPlan, PagedKV, Param, Part, Piece, StepShape
 from .registry import register
@@ -34,13 +43,22 @@ from .registry import register
 class DistanceBiasAttention(Part):
     def __init__(self, width: int, n_heads: int, n_kv_heads: int, dim: int, vdim: int, eps: float, scale: Optional[float] = None,
                  whole_qk_norm: bool = True, value_norm: bool = True, distance_bias: bool = True, chunk: Optional[int] = None,
-                 sink: Optional[float] = 0.0, window: Optional[int] = None):
+                 sink: Optional[float] = 0.0, window: Optional[int] = None, head_qk_norm: bool = False, log_bias: bool = False,
+                 learned_sink: bool = False, value_mix: Optional[str] = None, mix_key: str = "v_first"):
+        if (whole_qk_norm and head_qk_norm) or (distance_bias and log_bias) or (learned_sink and sink is not None):
+            raise ConfigError("distance_bias_attention: one kind of query/key norm, of distance bias and of sink at a time")
+        if value_mix not in (None, "first", "mix"):
+            raise ConfigError(f"distance_bias_attention: value_mix {value_mix!r} must be None, 'first' or 'mix'")
+        if (head_qk_norm or value_mix) and value_norm:
+            raise ConfigError("distance_bias_attention: a value norm is not built beside a norm per head or mixed values")
+        self.head_qk_norm, self.log_bias, self.learned_sink = head_qk_norm, log_bias, learned_sink
+        self.value_mix, self.mix_key = value_mix, mix_key
         self.width, self.n_heads, self.n_kv_heads, self.dim, self.vdim = width, n_heads, n_kv_heads, dim, vdim
         self.row = -(-max(dim, vdim) // 16) * 16         # a head in the cache and the kernels: padded with zeros
         self.eps, self.scale = float(eps), dim ** -0.5 if scale is None else float(scale)
         self.whole_qk_norm, self.value_norm, self.distance_bias = whole_qk_norm, value_norm, distance_bias
         self.chunk, self.sink, self.window = chunk, sink, window
-        self.proj_weight = self.q_norm = self.k_norm = self.o_weight = self.slopes = self.sinks = None
+        self.proj_weight = self.q_norm = self.k_norm = self.o_weight = self.slopes = self.sinks = self.rates = self.vmix = None
 
     def params(self) -> List[Param]:
         q, k, v = self.n_heads * self.dim, self.n_kv_heads * self.dim, self.n_kv_heads * self.vdim
@@ -50,6 +68,13 @@ class DistanceBiasAttention(Part):
         if self.whole_qk_norm:
             ps += [Param("q_norm", (Piece("q.norm", (q,)),), kind="vector", init="one_plus_normal"),
                    Param("k_norm", (Piece("k.norm", (k,)),), kind="vector", init="one_plus_normal")]
+        if self.log_bias:
+            ps += [Param("slopes", (Piece("r1", (self.n_heads,)),), kind="vector", init="const:0.5"),
+                   Param("rates", (Piece("r2", (self.n_heads,)),), kind="vector", init="const:0.5")]
+        if self.learned_sink:
+            ps.append(Param("sinks", (Piece("sink", (self.n_heads,)),), kind="vector"))
+        if self.value_mix:
+            ps.append(Param("vmix", (Piece("vmix", ()),), kind="vector", init="const:0.4"))
         return ps
 
     def assign(self, attr: str, tensor: torch.Tensor) -> None:
@@ -72,7 +97,7 @@ class DistanceBiasAttention(Part):
         return ("distance_bias_attention", self.n_heads, self.n_kv_heads, self.row, self.window, self.chunk)
 
     def plan(self, shape: StepShape) -> AttentionPlan:
-        splits = decode_splits(shape, self.n_kv_heads)
+        splits = decode_splits(shape, self.n_kv_heads, self.window)
         if self.chunk:                                           # no token reads more keys than a chunk holds: parts of
             while splits > 1 and splits * 512 > self.chunk:      # 512 keys at least
                 splits //= 2
@@ -84,8 +109,17 @@ class DistanceBiasAttention(Part):
         slots = gb.slots if cache.store else None
         H, G, d, dv, row = self.n_heads, self.n_kv_heads, self.dim, self.vdim, self.row
         proj = _linear(h, self.proj_weight)                      # [T, q | k | v]
-        q = ops.whole_norm_store(proj, 0, H * d, (H + G) * d, self.q_norm, self.k_norm, self.eps, self.value_norm, slots,
-                                 cache.k, cache.v, H, G, d, dv, row, cache.page_size)
+        if self.head_qk_norm or self.value_mix:
+            v_off, mix, first = (H + G) * d, None, None
+            if self.value_mix == "first":
+                batch.carry[self.mix_key] = proj[:, v_off:v_off + G * dv]
+            elif self.value_mix == "mix":
+                mix, first = self.vmix, batch.carry[self.mix_key]
+            q = ops.head_norm_store(proj, 0, H * d, v_off, self.head_qk_norm, self.eps, slots, cache.k, cache.v, H, G, d, dv, row,
+                                    cache.page_size, mix, first)
+        else:
+            q = ops.whole_norm_store(proj, 0, H * d, (H + G) * d, self.q_norm, self.k_norm, self.eps, self.value_norm, slots,
+                                     cache.k, cache.v, H, G, d, dv, row, cache.page_size)
         out = torch.empty((h.shape[0], H * row), dtype=h.dtype, device=h.device)
         plan = batch.plan(self)
         splits = plan.splits if plan is not None else 1
@@ -93,12 +127,12 @@ class DistanceBiasAttention(Part):
             ops.paged_attention_mma(q, cache.k, cache.v, out, batch.tok_seg, batch.positions, gb.block_table, batch.cu_q,
                                     batch.prefill_segs, batch.num_prefill_segs, batch.max_prefill_q, batch.decode_tokens,
                                     batch.num_decode_tokens, H, G, row, cache.page_size, self.window, self.scale, splits,
-                                    batch.scratch, None, None, cache.k_map2d, cache.v_map2d, 0, slopes=self.slopes,
-                                    chunk=self.chunk, sinks=self.sinks)
+                                    batch.scratch, cache.k_map, cache.v_map, cache.k_map2d, cache.v_map2d, 0, slopes=self.slopes,
+                                    chunk=self.chunk, sinks=self.sinks, rates=self.rates)
         else:       # float32, or sizes the tensor-core kernels do not take
             ops.paged_attention(q, cache.k, cache.v, out, batch.tok_seg, batch.positions, gb.block_table, H, G, row,
                                 cache.page_size, self.window, self.scale, splits, batch.scratch, slopes=self.slopes,
-                                chunk=self.chunk, sinks=self.sinks)
+                                chunk=self.chunk, sinks=self.sinks, rates=self.rates)
         return _linear(out, self.o_weight)
 
 

@@ -1,4 +1,5 @@
-"""Gated feed-forward: down( act(gate(h)) * up(h) ) with gate and up as one matrix.
+"""Gated feed-forward: down( act(gate(h)) * up(h) ) with gate and up as one matrix; or the capped form down( g
+sigmoid(1.702 g) (u + 1) ) with g = min(gate(h), limit), u = clamp(up(h), -limit, limit).
 
 pico_vllm/model.py:309-318 (fused gate_up projection, silu(gate) * up, down projection);
 the activation runs in float32 as in pico_vllm/kernels/swiglu.py:28-44.
@@ -19,10 +20,13 @@ from .registry import register
 class GatedMLP(Part):
     fuses_residual = True   # forward(..., residual=x) may add its output to x and return None
 
-    def __init__(self, width: int, inner: int, act: str = "silu"):
-        if act != "silu":
-            raise ConfigError(f"gated_mlp: activation {act!r} is not built (only 'silu')")
-        self.width, self.inner = width, inner
+    def __init__(self, width: int, inner: int, act: str = "silu", limit: Optional[float] = None):
+        if act not in ("silu", "capped"):
+            raise ConfigError(f"gated_mlp: activation {act!r} is not built (only 'silu' and 'capped')")
+        if (act == "capped") != bool(limit and limit > 0):
+            raise ConfigError("gated_mlp: the capped activation, and it alone, needs a positive limit")
+        self.width, self.inner, self.act = width, inner, act
+        self.limit = float(limit) if limit else None
         self.gate_up_weight = self.down_weight = None
 
     def params(self) -> List[Param]:
@@ -40,17 +44,20 @@ class GatedMLP(Part):
         With ``norm`` (after ``can_fuse_norm``), ``h`` is None and the normed input is computed from
         ``residual`` inside the first kernel."""
         if norm is not None:
-            a = ops.skinny_gate_up_swiglu(residual, self.gate_up_weight, norm.weight, norm.eps)
+            a = ops.skinny_gate_up_swiglu(residual, self.gate_up_weight, norm.weight, norm.eps, limit=self.limit)
         elif ops.skinny_takes(h, self.gate_up_weight) and self.inner % 8 == 0:
-            a = ops.skinny_gate_up_swiglu(h, self.gate_up_weight)      # product and activation in one kernel
+            a = ops.skinny_gate_up_swiglu(h, self.gate_up_weight, limit=self.limit)      # product and activation in one kernel
         elif h.shape[0] >= ops.TC_PAIR_MIN_TOKENS and ops.tc_takes(h, self.gate_up_weight) and self.inner % 8 == 0:
             # many tokens: tcgen05 product with the activation in its epilogue (the [T, 2I] buffer never exists);
             # below that the library product and the activation kernel are faster (measured, see ops)
-            a = ops.tc_gate_up_swiglu(h, self.gate_up_weight)
+            a = ops.tc_gate_up_swiglu(h, self.gate_up_weight, limit=self.limit)
         else:
             gu = ops.linear(h, self.gate_up_weight)
-            a = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
-            ops.swiglu(gu, a)
+            if self.limit:
+                a = ops.capped_glu(gu, self.inner, self.limit)
+            else:
+                a = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
+                ops.swiglu(gu, a)
         if residual is not None and ops.skinny_takes(a, self.down_weight):
             ops.skinny_linear_residual(a, self.down_weight, residual)
             return None

@@ -16,6 +16,7 @@ from typing import List, Optional, Union
 import torch
 
 from .. import ops
+from ..errors import ConfigError, KernelError
 from .base import Param, Part, Piece
 from .registry import register
 
@@ -35,6 +36,8 @@ class SumDelta:
     terms: list
 
     def flat(self):
+        if any(getattr(n, "groups", 1) != 1 for _, n, _ in self.terms):
+            raise KernelError("several outputs added together: norms in groups are not built")
         return [(d, None if n is None else n.weight, ops.NORM_NONE if n is None else n.norm_kind, 0.0 if n is None else n.eps, s)
                 for d, n, s in self.terms]
 
@@ -55,7 +58,8 @@ def _post_add_norm(norm, kind: int, x: torch.Tensor, delta, rows: Optional[torch
     if isinstance(delta, NormedDelta):
         post, delta = delta.norm, delta.delta
     return ops.post_add_norm(x, delta, None if post is None else post.weight, 0 if post is None else post.norm_kind,
-                             0.0 if post is None else post.eps, norm.weight, kind, norm.eps, out, rows)
+                             0.0 if post is None else post.eps, norm.weight, kind, norm.eps, out, rows,
+                             post_groups=getattr(post, "groups", 1), groups=getattr(norm, "groups", 1))
 
 
 @register("norm", "rmsnorm")
@@ -117,6 +121,27 @@ class ScalarRMSNorm(RMSNorm):
         setattr(self, attr, tensor)
 
 
+@register("norm", "grouped_rmsnorm")
+class GroupedRMSNorm(RMSNorm):
+    """The row in ``groups`` equal runs of neighbours, each divided by its own sqrt(mean(run^2) + eps); the whole times a weight
+    per coordinate.  One group: an RMS norm."""
+
+    def __init__(self, width: int, eps: float, groups: int = 1):
+        super().__init__(width, eps, one_plus=False)
+        if groups < 1 or width % groups:
+            raise ConfigError(f"grouped_rmsnorm: {groups} groups do not divide a width of {width} evenly")
+        self.groups = groups
+        self.plain_rms = groups == 1
+
+    def add_norm(self, x: torch.Tensor, delta: Union[None, torch.Tensor, NormedDelta],
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if self.groups > 1 and (x.dim() != 2 or isinstance(delta, SumDelta)):
+            raise KernelError("grouped_rmsnorm: built for one residual stream and one output added at a time")
+        if self.groups == 1:
+            return super().add_norm(x, delta, rows)
+        return _post_add_norm(self, ops.NORM_RMS, x, delta, rows)
+
+
 @register("norm", "centred_norm")
 class CentredNorm(Part):
     """y = (x - mean x) / sqrt(mean((x - mean x)^2) + eps) * weight: a layer norm with a weight and no bias,
@@ -166,6 +191,7 @@ class PassNorm(Part):
                 post, delta = delta.norm, delta.delta
             if delta is not None:
                 ops.post_add_norm(x, delta, None if post is None else post.weight, 0 if post is None else post.norm_kind,
-                                  0.0 if post is None else post.eps, None, ops.NORM_NONE, 0.0, None, None)
+                                  0.0 if post is None else post.eps, None, ops.NORM_NONE, 0.0, None, None,
+                                  post_groups=getattr(post, "groups", 1))
             return x
         return _post_add_norm(self, ops.NORM_COPY, x, delta, rows)

@@ -54,6 +54,9 @@ def _register_builtin() -> None:
     from .config.banazen import BanazenConfig
     from .models.banazen import build_banazen
     register_architecture("Banazen", BanazenConfig, build_banazen)
+    from .config.vanapel import VanapelConfig
+    from .models.vanapel import build_vanapel
+    register_architecture("Vanapel", VanapelConfig, build_vanapel)
 
 
 _register_builtin()

@@ -77,7 +77,7 @@ def attention_scratch_floats(T, n_heads, head_dim, n_splits):
 
 def paged_attention(q, k_pages, v_pages, out, tok_seg, positions, block_table, n_heads, n_kv_heads,
                     head_dim, page_size, window, scale, n_splits=1, scratch=None, softcap=None, slopes=None, chunk=None,
-                    sinks=None):
+                    sinks=None, rates=None):
     T = q.shape[0]
     g = n_heads // n_kv_heads
     for t in range(T):
@@ -98,7 +98,8 @@ def paged_attention(q, k_pages, v_pages, out, tok_seg, positions, block_table, n
             if softcap:
                 s = softcap * torch.tanh(s / softcap)
             if slopes is not None:
-                s = s - float(slopes[h]) * (p - n).float()
+                dist = (p - n).float()
+                s = s - float(slopes[h]) * (dist if rates is None else torch.log1p(float(rates[h]) * dist))
             if sinks is not None:
                 e = torch.exp(s - float(sinks[h]))
                 pr = e / (1.0 + e.sum())
@@ -116,9 +117,9 @@ def mma_attention_takes(dtype, n_heads, n_kv_heads, head_dim):
 def paged_attention_mma(q, k_pages, v_pages, out, tok_seg, positions, block_table, cu_q, prefill_segs,
                         n_prefill_segs, max_prefill_q, decode_tokens, n_decode_tokens, n_heads, n_kv_heads, head_dim,
                         page_size, window, scale, n_splits=1, scratch=None, k_map=None, v_map=None, k_map2d=None,
-                        v_map2d=None, pair_min_keys=0, softcap=None, slopes=None, chunk=None, sinks=None):
+                        v_map2d=None, pair_min_keys=0, softcap=None, slopes=None, chunk=None, sinks=None, rates=None):
     return paged_attention(q, k_pages, v_pages, out, tok_seg, positions, block_table, n_heads, n_kv_heads, head_dim,
-                           page_size, window, scale, softcap=softcap, slopes=slopes, chunk=chunk, sinks=sinks)
+                           page_size, window, scale, softcap=softcap, slopes=slopes, chunk=chunk, sinks=sinks, rates=rates)
 
 
 SKINNY_MAX_TOKENS = 16
@@ -161,12 +162,12 @@ def skinny_linear_residual(x, weight, residual):
     residual.add_(x.float() @ weight.float().t())
 
 
-def skinny_gate_up_swiglu(x, gate_up_weight, norm_weight=None, eps=0.0):
+def skinny_gate_up_swiglu(x, gate_up_weight, norm_weight=None, eps=0.0, limit=None):
     x = _normed(x, norm_weight, eps)
     gu = x.float() @ gate_up_weight.float().t()
     I = gu.shape[1] // 2
     g, u = gu[:, :I], gu[:, I:]
-    return (g * torch.sigmoid(g) * u).to(torch.bfloat16)
+    return (_capped(g, u, limit) if limit else g * torch.sigmoid(g) * u).to(torch.bfloat16)
 
 
 def skinny_qkv_rope_store(x, qkv_weight, bias, positions, inv_freq, slots, k_pages, v_pages, n_heads, n_kv_heads,
@@ -220,17 +221,22 @@ def sample(logits, temperature, top_p, uniform, out):
 
 
 # ------------------------------------------------------------------ norm -> add -> norm, latent attention, routed experts
-def _norm(u, kind, w, eps):
+def _norm(u, kind, w, eps, groups=1):
     if kind in (0, 3):          # none; 3: no norm on the way out, the row is only written in the activation type
         return u
+    if groups > 1:              # equal runs of the row, a root mean square each
+        runs = u.view(u.shape[0], groups, -1)
+        y = (runs / torch.sqrt((runs * runs).mean(-1, keepdim=True) + eps)).view(u.shape)
+        return y if w is None else y * w
     if kind == 2:
         u = u - u.mean(-1, keepdim=True)
     y = u / torch.sqrt((u * u).mean(-1, keepdim=True) + eps)
     return y if w is None else y * w
 
 
-def post_add_norm(x, delta, post_weight, post_kind, post_eps, weight, kind, eps, out, rows=None):
-    d = None if delta is None else _norm(delta.float(), post_kind, post_weight, post_eps)
+def post_add_norm(x, delta, post_weight, post_kind, post_eps, weight, kind, eps, out, rows=None, post_groups=1,
+                  groups=1):
+    d = None if delta is None else _norm(delta.float(), post_kind, post_weight, post_eps, post_groups)
     if rows is None:
         if d is not None:
             x.add_(d)
@@ -240,7 +246,7 @@ def post_add_norm(x, delta, post_weight, post_kind, post_eps, weight, kind, eps,
         if d is not None:
             src = src + d[rows.long()]
     if out is not None:
-        out.copy_(_norm(src, kind, weight, eps).to(out.dtype))
+        out.copy_(_norm(src, kind, weight, eps, groups).to(out.dtype))
     return out
 
 
@@ -251,7 +257,7 @@ def scale_softcap(logits, scale, cap):
     return logits
 
 
-def latent_norm_store(proj, q_off, q_rank, q_weight, kv_off, kv_rank, kv_weight, slots, cache, g_off, heads, eps):
+def latent_norm_store(proj, q_off, q_rank, q_weight, kv_off, kv_rank, kv_weight, slots, cache, g_off, heads, eps, rot=None):
     p = proj.float()
     cq = _norm(p[:, q_off:q_off + q_rank], 1, q_weight, eps).to(proj.dtype) if q_rank > 0 else None
     if kv_rank > 0:
@@ -261,7 +267,47 @@ def latent_norm_store(proj, q_off, q_rank, q_weight, kv_off, kv_rank, kv_weight,
             if s >= 0:
                 flat[s].zero_()
                 flat[s, :kv_rank] = c[t]
+        if rot is not None:
+            off, dim, positions, inv_freq, mult = rot
+            kr = rotate_tail(p[:, off:off + dim].clone(), 1, dim, positions, inv_freq, mult)
+            for t, s in enumerate(slots.tolist()):
+                if s >= 0:
+                    flat[s, kv_rank:kv_rank + dim] = kr[t].to(cache.dtype)
     return cq, (torch.sigmoid(p[:, g_off:g_off + heads]) if heads > 0 else None)
+
+
+def rotate_tail(x, heads, rot_dim, positions, inv_freq, mult=1.0):
+    T, half = x.shape[0], inv_freq.shape[0]
+    v = x.view(T, heads, -1)[..., -rot_dim:]
+    a = positions.float()[:, None] * inv_freq[None, :]
+    c, s = (torch.cos(a) * mult)[:, None, :], (torch.sin(a) * mult)[:, None, :]
+    u, w = v[..., :half].float(), v[..., half:2 * half].float()
+    keep = (positions < 0)[:, None, None]
+    v1, v2 = torch.where(keep, u, u * c - w * s), torch.where(keep, w, w * c + u * s)
+    v[..., :half], v[..., half:2 * half] = v1.to(x.dtype), v2.to(x.dtype)
+    return x
+
+
+def head_norm_store(proj, q_off, k_off, v_off, norm, eps, slots, k_pages, v_pages, heads, kv_heads, dim, vdim, row, page_size,
+                    mix=None, first=None):
+    T = proj.shape[0]
+    p = proj.float()
+    q = p[:, q_off:q_off + heads * dim].reshape(T, heads, dim)
+    k = p[:, k_off:k_off + kv_heads * dim].reshape(T, kv_heads, dim)
+    v = p[:, v_off:v_off + kv_heads * vdim].reshape(T, kv_heads, vdim)
+    if norm:
+        q, k = _rms_unit(q, eps), _rms_unit(k, eps)
+    if mix is not None:
+        v = (1.0 - float(mix)) * v + float(mix) * first.float().reshape(T, kv_heads, vdim)
+    pad = lambda t, d: torch.cat([t, torch.zeros(t.shape[0], t.shape[1], row - d)], 2)
+    q, k, v = pad(q, dim), pad(k, dim), pad(v, vdim)
+    if slots is not None:
+        for t in range(T):
+            sl = int(slots[t])
+            if sl >= 0:
+                k_pages[sl // page_size, :, sl % page_size, :] = k[t].to(k_pages.dtype)
+                v_pages[sl // page_size, :, sl % page_size, :] = v[t].to(v_pages.dtype)
+    return q.reshape(T, heads * row).to(proj.dtype)
 
 
 def head_linear(x, weight, out, gate=None):
@@ -563,7 +609,7 @@ def whole_norm_store(proj, q_off, k_off, v_off, q_w, k_w, eps, v_norm, slots, k_
     return q.reshape(T, heads * row).to(proj.dtype)
 
 
-NAMES = ["hyper_expand", "hyper_step", "scale_add_rows", "scaled_sum", "gated_linear_attention", "mlstm_prepare", "hgrn2_prepare",
+NAMES = ["rotate_tail", "head_norm_store", "hyper_expand", "hyper_step", "scale_add_rows", "scaled_sum", "gated_linear_attention", "mlstm_prepare", "hgrn2_prepare",
          "causal_conv_silu", "mamba2_prepare", "group_rms_norm", "whole_norm_store",
          "activation", "qk_norm_rope_store", "sigmoid_gate", "decay_linear_attention", "gated_rms_norm", "post_add_norm", "scale_softcap", "latent_norm_store", "head_linear", "head_scale", "moe_route", "moe_experts",
          "embedding", "add_rmsnorm", "swiglu", "rope_store", "attention_scratch_floats", "paged_attention",
