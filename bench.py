@@ -615,8 +615,26 @@ def banazen_config(shape, layers):
                 logit_scale=1.0, token_side=dict(dim=64), layers=zl)
 
 
-# the model a design is measured beside: the closest one the package had before it
-DESIGN_BESIDE = {"zapipel": "qwen2", "zikupel": "qwen2", "zazilix": "zikupel", "banazen": "zazilix"}
+def vanapel_config(shape, layers):
+    """The Vanapel design at the sizes of ``shape``, norms in two groups: three layers of softmax attention over a window of
+    1,024 positions (heads of the head size on the shape's key/value heads, values mixed with the first layer's) to one of
+    latent attention (a quarter of every head rotated with stretched frequencies; latent and rotated key part together as wide
+    as the shape's latent); the capped dense feed-forward in every layer."""
+    s = DESIGN_SHAPES[shape]
+    H, d = s["heads"], s["head"]
+    att = dict(heads=H, kv_heads=s["kv_heads"], dim=d, vdim=d, scale=d ** -0.5, mask=dict(size=1024), v_mix=True)
+    lat = dict(heads=H, dim=d * 3 // 4, rot_dim=d // 4, vdim=d, q_rank=s["q_rank"], kv_rank=s["kv_rank"] - d // 4, scale=d ** -0.5,
+               rot=dict(base=10000.0, dims=d // 4, scaling=dict(factor=8.0, original=1024, fast=16.0, slow=2.0)))
+    mlp = dict(kind="dense", ff=s["ff"], limit=7.0)
+    zl = [dict(type="latent_attention" if i % 4 == 3 else "attention", mixer=dict(lat if i % 4 == 3 else att), mlp=mlp)
+          for i in range(layers)]
+    return dict(architecture="Vanapel", vocab=DESIGN_VOCAB, width=s["width"], norm=dict(eps=1e-5, groups=2), layers=zl)
+
+
+# the models a design is measured beside: the closest ones the package had before it (zapipel_dense: the Zapipel design with
+# latents of its own and the dense feed-forward in every layer)
+DESIGN_BESIDE = {"zapipel": ["qwen2"], "zikupel": ["qwen2"], "zazilix": ["zikupel"], "banazen": ["zazilix"],
+                 "vanapel": ["zapipel_dense", "qwen2"]}
 
 
 def design_configs(shape, layers):
@@ -633,16 +651,17 @@ def design_configs(shape, layers):
                                     router=dict(experts=s["experts"], top=s["top"]))))
     zap = dict(architecture="Zapipel", vocab=DESIGN_VOCAB, width=s["width"], norm=dict(eps=1e-5), logit_scale=1.0,
                logit_softcap=30.0, layers=zl)
+    zap_dense = dict(zap, layers=[dict(type="latent_attention", mixer=dict(mixer), mlp=dict(kind="dense", ff=s["ff"]))] * layers)
     qwen = dict(MODEL, vocab_size=DESIGN_VOCAB, hidden_size=s["width"], num_hidden_layers=layers,
                 num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=s["head"],
                 intermediate_size=s["ff"], tie_word_embeddings=False)
     return {"zapipel": zap, "qwen2": qwen, "zikupel": zikupel_config(shape, layers), "zazilix": zazilix_config(shape, layers),
-            "banazen": banazen_config(shape, layers)}
+            "banazen": banazen_config(shape, layers), "vanapel": vanapel_config(shape, layers), "zapipel_dense": zap_dense}
 
 
 def run_design(args):
     """Prefill (one 2,048-token prompt) and decode (``--batch`` requests at ``--context``; default 8 and 64 at
-    2,048) of the named design and of the Qwen2 decoder at equal sizes, random weights drawn on the device.
+    2,048) of the named design and of the models it is measured beside at equal sizes, random weights drawn on the device.
     Prints one JSON line; with ``--only`` and ``--arch`` one phase of one model (for a launch list)."""
     import torch
     import pico_vllm_b200  # noqa: F401
@@ -652,7 +671,7 @@ def run_design(args):
     context = args.context or 2048
     batches = [args.batch] if args.batch else [8, 64]
     shapes = sorted(DESIGN_SHAPES) if args.shape == "all" else [args.shape]
-    archs = [args.design, DESIGN_BESIDE[args.design]] if args.arch == "both" else [args.arch]
+    archs = [args.design] + DESIGN_BESIDE[args.design] if args.arch == "both" else [args.arch]
     out = {"design": args.design, "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random weights N(0, 0.02)",
            "layers": layers, "vocab": DESIGN_VOCAB, "context": context, "peaks": pk["source"], "shapes": {}}
     sampler = ClockSampler()
@@ -792,12 +811,13 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 and 64")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one phase only and print a short line (for profiling; not a bench value)")
-    ap.add_argument("--design", choices=["zapipel", "zikupel", "zazilix", "banazen"], default=None,
+    ap.add_argument("--design", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel"], default=None,
                     help="the named design beside the closest earlier model at equal sizes (zapipel, zikupel: the Qwen2 decoder; "
-                         "zazilix: zikupel; banazen: zazilix), prefill and decode; not the default run")
+                         "zazilix: zikupel; banazen: zazilix; vanapel: zapipel with dense layers, and the Qwen2 decoder), "
+                         "prefill and decode; not the default run")
     ap.add_argument("--shape", choices=sorted(DESIGN_SHAPES) + ["all"], default="all", help="with --design: which sizes")
-    ap.add_argument("--arch", choices=["zapipel", "zikupel", "zazilix", "banazen", "qwen2", "both"], default="both",
-                    help="with --design: which model (both: the design and the model it is measured beside)")
+    ap.add_argument("--arch", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel", "zapipel_dense", "qwen2", "both"],
+                    default="both", help="with --design: which model (both: the design and what it is measured beside)")
     ap.add_argument("--micro", action="store_true",
                     help="time single decode kernels replayed from a graph (skinny products, decode attention)")
     ap.add_argument("--profile-range", choices=["decode", "prefill"], default=None,
