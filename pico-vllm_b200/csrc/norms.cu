@@ -175,25 +175,32 @@ __global__ void post_add_norm_kernel(float* __restrict__ x, const TA* __restrict
 // The same work with a warp per row and the row in registers (H a multiple of 4, at most 128 * VPL elements): every
 // load of a row - what is added and the stream - is issued before anything is waited for, the sums
 // go through shuffles, and nothing passes through shared memory or a block barrier.  Four rows a block.
-// GROUPED: `groups` equal runs of H / groups elements (a multiple of 4), a root mean square each.
-template <int VPL, bool GROUPED>
+// GROUPED: `groups` equal runs of H / groups elements (a multiple of 4), a root mean square each; 1: one or two runs, 2: any number
+// (the vectors that lie outside the runs at hand are passed over), 0: one root mean square.
+template <int VPL, int GROUPED>
 __device__ __forceinline__ void norm_regs(float4 (&v)[VPL], const float* __restrict__ w, int n4, int lane, int H, int kind,
                                           float eps, int groups) {
-    if (GROUPED && groups > 1) {
+    if (GROUPED != 0 && groups > 1) {
         const int gn = n4 / groups;
-        for (int g = 0; g < groups; ++g) {
-            const int lo = g * gn, hi = lo + gn;
-            float gs = 0.f;
+        for (int g = 0; g < groups; g += 2) {            // two groups at a time: their sums' exchanges run side by side
+            const int lo = g * gn, mid = lo + gn, hi = g + 1 < groups ? mid + gn : mid;
+            float s0 = 0.f, s1 = 0.f;
 #pragma unroll
             for (int k = 0; k < VPL; ++k) {
+                if (GROUPED == 2 && (32 * k >= hi || 32 * k + 32 <= lo)) continue;      // none of the warp's vectors lies in the two groups
                 const int i = lane + 32 * k;
-                if (i >= lo && i < hi) gs += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+                const float sq = (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+                s0 += i >= lo && i < mid ? sq : 0.f;
+                s1 += i >= mid && i < hi ? sq : 0.f;
             }
-            const float ginv = 1.0f / sqrtf(warp_sum(gs) / (float)(4 * gn) + eps);
+            const float len = (float)(4 * gn);
+            const float inv0 = 1.0f / sqrtf(warp_sum(s0) / len + eps), inv1 = 1.0f / sqrtf(warp_sum(s1) / len + eps);
 #pragma unroll
             for (int k = 0; k < VPL; ++k) {
+                if (GROUPED == 2 && (32 * k >= hi || 32 * k + 32 <= lo)) continue;
                 const int i = lane + 32 * k;
-                if (i >= lo && i < hi) { v[k].x *= ginv; v[k].y *= ginv; v[k].z *= ginv; v[k].w *= ginv; }
+                const float inv = i < lo || i >= hi ? 1.0f : i < mid ? inv0 : inv1;
+                v[k].x *= inv; v[k].y *= inv; v[k].z *= inv; v[k].w *= inv;
             }
         }
         if (!w) return;
@@ -232,8 +239,9 @@ __device__ __forceinline__ void norm_regs(float4 (&v)[VPL], const float* __restr
     }
 }
 
-template <typename TA, int VPL, bool GROUPED>
-__global__ void __launch_bounds__(128) post_add_norm_warp_kernel(float* __restrict__ x, const TA* __restrict__ delta,
+// GROUPED rows of up to 1,536 keep four blocks on a multiprocessor: 2,048 of them are then one wave, as without groups.
+template <typename TA, int VPL, int GROUPED>
+__global__ void __launch_bounds__(128, GROUPED == 0 ? 1 : VPL <= 12 ? 4 : 2) post_add_norm_warp_kernel(float* __restrict__ x, const TA* __restrict__ delta,
                                                                  const float* __restrict__ post_w, int post_kind,
                                                                  float post_eps, const float* __restrict__ w, int kind,
                                                                  float eps, TA* __restrict__ out,
@@ -271,7 +279,7 @@ __global__ void __launch_bounds__(128) post_add_norm_warp_kernel(float* __restri
         if (lane + 32 * k < n4) Row4<TA>::store(dst + 4 * (lane + 32 * k), a[k]);
 }
 
-template <typename TA, bool GROUPED>
+template <typename TA, int GROUPED>
 static void launch_pan_warp(int vpl, dim3 grid, cudaStream_t stream, float* x, const void* delta, const float* post_w,
                             int post_kind, float post_eps, const float* w, int kind, float eps, void* out, const int* rows,
                             int R, int H, int post_groups, int groups) {
@@ -297,7 +305,7 @@ PICO_API int pico_post_add_norm(float* x, const void* delta, const float* post_w
     if (post_groups < 1 || groups < 1 || H % post_groups || H % groups || (post_groups > 1 && post_kind == NORM_CENTRED) ||
         (groups > 1 && kind == NORM_CENTRED))
         return PICO_ERR_SIZE;
-    const bool grouped = post_groups > 1 || groups > 1;
+    const int most = post_groups > groups ? post_groups : groups, grouped = most > 2 ? 2 : most > 1 ? 1 : 0;
     const bool v4 = H % 4 == 0 && (H / post_groups) % 4 == 0 && (H / groups) % 4 == 0;      // a vector lies within one group
     if (post_kind < 0 || post_kind > 2 || kind < 0 || kind > 3) return PICO_ERR_SIZE;
     if (act_dtype != PICO_F32 && act_dtype != PICO_BF16) return PICO_ERR_DTYPE;
@@ -308,9 +316,9 @@ PICO_API int pico_post_add_norm(float* x, const void* delta, const float* post_w
     launch_pan_warp<TA, GR>(vpl, grid, stream, x, delta, post_w, post_kind, post_eps, w, kind, eps, out, rows, R, H,       \
                             post_groups, groups)
         if (act_dtype == PICO_F32) {
-            if (grouped) PAN_ROWS(float, true); else PAN_ROWS(float, false);
+            if (grouped == 2) PAN_ROWS(float, 2); else if (grouped == 1) PAN_ROWS(float, 1); else PAN_ROWS(float, 0);
         } else {
-            if (grouped) PAN_ROWS(bf16, true); else PAN_ROWS(bf16, false);
+            if (grouped == 2) PAN_ROWS(bf16, 2); else if (grouped == 1) PAN_ROWS(bf16, 1); else PAN_ROWS(bf16, 0);
         }
 #undef PAN_ROWS
         return pico_launch_status();
