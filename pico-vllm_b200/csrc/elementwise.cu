@@ -203,3 +203,64 @@ PICO_API int pico_swiglu(const void* gate_up, void* out, int T, int I, int act_d
         return PICO_ERR_DTYPE;
     return pico_launch_status();
 }
+
+// ---------------------------------------------------------------- gated activation with biases
+// gate_up [T, 2*I] with the gate columns first; g = gate + bias[i], u = up + bias[I + i] (bias float32 [2*I] or nullptr);
+// out[t, i] = act(g) * u.  act: 0 silu(g) = g / (1 + e^-g); 1 the tanh form of gelu, g / 2 (1 + tanh(z)) with
+// z = sqrt(2 / pi) (g + 0.044715 g^3), computed as g / (1 + e^(-2 z)).
+__device__ __forceinline__ float bg_act(float g, int act) {
+    const float z = act == 1 ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+    return g / (1.0f + expf(-z));
+}
+
+// W: 8 (bfloat16, I a multiple of 8, 16 bytes per access) or 1.
+template <typename TA, int W>
+__global__ void bias_glu_kernel(const TA* __restrict__ gate_up, const float* __restrict__ bias, int act, TA* __restrict__ out,
+                                int I, size_t items) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int per = I / W;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < items; idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = idx / per;
+        const int i = (int)(idx - t * per) * W;
+        const TA* row = gate_up + t * 2 * (size_t)I;
+        if constexpr (W == 1) {
+            const float g = to_f32(row[i]) + (bias ? bias[i] : 0.f), u = to_f32(row[I + i]) + (bias ? bias[I + i] : 0.f);
+            out[idx] = from_f32<TA>(bg_act(g, act) * u);
+        } else {
+            const uint4 graw = *reinterpret_cast<const uint4*>(row + i), uraw = *reinterpret_cast<const uint4*>(row + I + i);
+            const TA* g = reinterpret_cast<const TA*>(&graw);
+            const TA* u = reinterpret_cast<const TA*>(&uraw);
+            float bg[W], bu[W];
+#pragma unroll
+            for (int k = 0; k < W; k += 4) {
+                const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+                *reinterpret_cast<float4*>(bg + k) = bias ? *reinterpret_cast<const float4*>(bias + i + k) : z;
+                *reinterpret_cast<float4*>(bu + k) = bias ? *reinterpret_cast<const float4*>(bias + I + i + k) : z;
+            }
+            uint4 res;
+            TA* o = reinterpret_cast<TA*>(&res);
+#pragma unroll
+            for (int k = 0; k < W; ++k) o[k] = from_f32<TA>(bg_act(to_f32(g[k]) + bg[k], act) * (to_f32(u[k]) + bu[k]));
+            *reinterpret_cast<uint4*>(out + t * (size_t)I + i) = res;
+        }
+    }
+}
+
+PICO_API int pico_bias_glu(const void* gate_up, const float* bias, int act, void* out, int T, int I, int dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (I < 1 || (act != 0 && act != 1)) return PICO_ERR_SIZE;
+    const bool vec = dtype == PICO_BF16 && I % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out | (uintptr_t)bias) & 15) == 0;
+    const size_t items = (size_t)T * (vec ? I / 8 : I), want = (items + 255) / 256;
+    const long long cap = 16LL * pico_num_sms();
+    const dim3 grid((unsigned)((long long)want > cap ? cap : (long long)want));
+    if (vec)
+        pico_launch((bias_glu_kernel<bf16, 8>), grid, dim3(256), 0, stream, (const bf16*)gate_up, bias, act, (bf16*)out, I, items);
+    else if (dtype == PICO_BF16)
+        pico_launch((bias_glu_kernel<bf16, 1>), grid, dim3(256), 0, stream, (const bf16*)gate_up, bias, act, (bf16*)out, I, items);
+    else if (dtype == PICO_F32)
+        pico_launch((bias_glu_kernel<float, 1>), grid, dim3(256), 0, stream, (const float*)gate_up, bias, act, (float*)out, I, items);
+    else
+        return PICO_ERR_DTYPE;
+    return pico_launch_status();
+}

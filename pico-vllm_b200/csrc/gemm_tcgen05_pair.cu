@@ -31,8 +31,8 @@
 #define TP_THREADS 192
 #define TP_WAIT_LIMIT (1 << 14)      // polls of a barrier (some microseconds each) before a thread gives up
 
-enum { TP_STORE = 0, TP_RESIDUAL = 1, TP_SWIGLU = 2, TP_CAPPED = 3 };
-__host__ __device__ constexpr bool tp_is_glu(int epi) { return epi == TP_SWIGLU || epi == TP_CAPPED; }
+enum { TP_STORE = 0, TP_RESIDUAL = 1, TP_SWIGLU = 2, TP_CAPPED = 3, TP_GELU = 4 };
+__host__ __device__ constexpr bool tp_is_glu(int epi) { return epi == TP_SWIGLU || epi == TP_CAPPED || epi == TP_GELU; }
 
 __device__ int g_tp_status = 0;
 PICO_API int pico_tp_status(int* out) {
@@ -110,6 +110,7 @@ struct TpArgs {
     bf16* out;                // STORE: [M, N]; SWIGLU: [M, N / 2]
     float* resid;             // RESIDUAL: [M, N]
     float limit;              // CAPPED: as SWIGLU with g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
+    const float* bias;        // GELU: as SWIGLU with gelu_tanh(g + bias[i]) * (u + bias[I + i]); float32 [N], or null
 };
 
 __device__ __forceinline__ void tp_st32(void* p, const uint32_t (&r)[8]) {      // one 32-byte store (a whole sector)
@@ -135,8 +136,15 @@ __device__ __forceinline__ float tp_capped_mul(float g, float u, float limit) {
     asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.0f + e));
     return g * r * (u + 1.0f);
 }
+// gelu_tanh(g) * u = g * u / (1 + 2^(-2 z log2 e)), z = sqrt(2 / pi) (g + 0.044715 g^3)
+__device__ __forceinline__ float tp_gelu_mul(float g, float u) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(fmaf(0.044715f * g * g, g, g) * (-1.5957691216057308f * 1.4426950408889634f)));
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.0f + e));
+    return g * r * u;
+}
 template <int EPI> __device__ __forceinline__ float tp_glu(float g, float u, float limit) {
-    return EPI == TP_CAPPED ? tp_capped_mul(g, u, limit) : tp_silu_mul(g, u);
+    return EPI == TP_GELU ? tp_gelu_mul(g, u) : EPI == TP_CAPPED ? tp_capped_mul(g, u, limit) : tp_silu_mul(g, u);
 }
 __device__ __forceinline__ uint32_t tp_pack(float a, float b) {
     __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -278,6 +286,21 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid
                     tp_ld32(taddr + c, g);
                     tp_ld32(taddr + BN / 2 + c, u);
                     asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+                    if (EPI == TP_GELU && p.bias) {            // the same columns for every lane: one transaction a load
+#pragma unroll
+                        for (int i = 0; i < 32; i += 4) {
+                            const int col = n0 + c + i;        // I is a multiple of 8: four columns are inside together or not at all
+                            if (col < I) {
+                                const float4 bg = *reinterpret_cast<const float4*>(p.bias + col), bu = *reinterpret_cast<const float4*>(p.bias + I + col);
+                                const float gb[4] = {bg.x, bg.y, bg.z, bg.w}, ub[4] = {bu.x, bu.y, bu.z, bu.w};
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    g[i + e] = __float_as_uint(__uint_as_float(g[i + e]) + gb[e]);
+                                    u[i + e] = __float_as_uint(__uint_as_float(u[i + e]) + ub[e]);
+                                }
+                            }
+                        }
+                    }
                     if (row < p.M) {
                         bf16* dst = p.out + (size_t)row * I + n0 + c;
 #pragma unroll
@@ -450,17 +473,19 @@ static void tp_pick(int M, int n_out, bool swiglu, int force_mb, int& bn_out, in
 }
 
 // epi: 0 = out[M, N] = x w^T (bfloat16); 1 = resid[M, N] (float32) += x w^T; 2 = out[M, N/2] =
-// silu(x wg^T) * (x wu^T) with w = [wg; wu]; 3 = the same with the capped form of the two products (limit > 0).  x: [M, K] bfloat16 with row stride ldx; w: [N, K] contiguous.
+// silu(x wg^T) * (x wu^T) with w = [wg; wu]; 3 = the same with the capped form of the two products (limit > 0); 4 = gelu_tanh(x wg^T + bg) * (x wu^T + bu) with bias = [bg; bu]
+// float32 (16-byte aligned) or nullptr.  x: [M, K] bfloat16 with row stride ldx; w: [N, K] contiguous.
 // rows_per_pair: 0 = chosen here, 256 or 512.
 PICO_API int pico_gemm_tcgen05_pair(const void* x, int ldx, const void* w, void* out, float* resid, int M, int N, int K,
-                                    int epi, int rows_per_pair, float limit, cudaStream_t stream) {
+                                    int epi, int rows_per_pair, float limit, const float* bias, cudaStream_t stream) {
     if (M < 1 || N < 16 || K < 16 || K % 8 != 0 || ldx % 8 != 0) return PICO_ERR_SIZE;
     if (epi == TP_CAPPED && !(limit > 0.f)) return PICO_ERR_SIZE;
+    if (epi < 0 || epi > TP_GELU || ((uintptr_t)bias & 15) != 0) return PICO_ERR_SIZE;
     if (tp_is_glu(epi) && (N % 2 != 0 || (N / 2) % 8 != 0)) return PICO_ERR_SIZE;
     if (!tp_is_glu(epi) && N % 8 != 0) return PICO_ERR_SIZE;
     if (rows_per_pair != 0 && rows_per_pair != 256 && rows_per_pair != 512) return PICO_ERR_SIZE;
     TpArgs a;
-    a.M = M; a.N = N; a.K = K; a.out = (bf16*)out; a.resid = resid; a.limit = limit;
+    a.M = M; a.N = N; a.K = K; a.out = (bf16*)out; a.resid = resid; a.limit = limit; a.bias = bias;
     int bn = 256, mb = 1;
     tp_pick(M, tp_is_glu(epi) ? N / 2 : N, tp_is_glu(epi), rows_per_pair / 256, bn, mb);
 #define TP_CASE(BN, MB)                                                                       \
@@ -469,6 +494,7 @@ PICO_API int pico_gemm_tcgen05_pair(const void* x, int ldx, const void* w, void*
         if (epi == TP_RESIDUAL) return tp_launch<BN, TP_RESIDUAL, MB>(x, ldx, w, a, stream);  \
         if (epi == TP_SWIGLU) return tp_launch<BN, TP_SWIGLU, MB>(x, ldx, w, a, stream);      \
         if (epi == TP_CAPPED) return tp_launch<BN, TP_CAPPED, MB>(x, ldx, w, a, stream);      \
+        if (epi == TP_GELU) return tp_launch<BN, TP_GELU, MB>(x, ldx, w, a, stream);          \
     }
     TP_CASE(256, 2)
     TP_CASE(256, 1)

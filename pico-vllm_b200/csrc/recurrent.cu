@@ -638,13 +638,14 @@ PICO_API int pico_mamba2_prepare(const void* proj, int row_stride, int dt_off, c
 //   den_floor:  val /= max(|x[t, g * group_stride + n]|, den_floor[t, g]) + 1e-6      (the normaliser rides as column n)
 //   skip:       val += skip_w[col / skip_head] * skip[t, col]
 //   pre_gate:   val *= silu(pre_gate[t, col])
-//   y[t, col] = val / sqrt(mean_j val^2 + eps) * w[col] * sigmoid(post_gate[t, col])       (w, post_gate optional)
+//   y[t, col] = val / sqrt(mean_j val^2 + eps) * w[col] * f(post_gate[t, col])       (w, post_gate optional; f is the sigmoid,
+//               or with post_act silu)
 template <typename TA, bool WIDE>
 __global__ void __launch_bounds__(256)
 group_rms_norm_kernel(const float* __restrict__ x, int x_stride, int group_stride, int groups, int n, const float* __restrict__ w,
                       float eps, const float* __restrict__ den_floor, const float* __restrict__ skip, int skip_stride,
                       const float* __restrict__ skip_w, int skip_head, const TA* __restrict__ pre_gate, int pre_stride,
-                      const TA* __restrict__ post_gate, int post_stride, TA* __restrict__ y) {
+                      const TA* __restrict__ post_gate, int post_stride, int post_act, TA* __restrict__ y) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
@@ -673,7 +674,10 @@ group_rms_norm_kernel(const float* __restrict__ x, int x_stride, int group_strid
         for (int j = tid; j < n; j += nth) {
             const int col = g * n + j;
             float o = value(j) * inv * (w ? w[col] : 1.0f);
-            if (post_gate) o *= rc_sigmoid(to_f32(post_gate[t * post_stride + col]));
+            if (post_gate) {
+                const float z = to_f32(post_gate[t * post_stride + col]);
+                o *= post_act ? rc_silu(z) : rc_sigmoid(z);
+            }
             y[t * ((size_t)groups * n) + col] = from_f32<TA>(o);
         }
     }
@@ -681,8 +685,8 @@ group_rms_norm_kernel(const float* __restrict__ x, int x_stride, int group_strid
 
 PICO_API int pico_group_rms_norm(const float* x, int x_stride, int group_stride, int groups, int n, const float* w, float eps,
                                  const float* den_floor, const float* skip, int skip_stride, const float* skip_w, int skip_head,
-                                 const void* pre_gate, int pre_stride, const void* post_gate, int post_stride, void* y, int T,
-                                 int dtype, cudaStream_t stream) {
+                                 const void* pre_gate, int pre_stride, const void* post_gate, int post_stride, int post_act, void* y,
+                                 int T, int dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (groups < 1 || n < 1 || (skip && (!skip_w || skip_head < 1))) return PICO_ERR_SIZE;
     if (groups > 65535 * 4) return PICO_ERR_SIZE;
@@ -691,7 +695,7 @@ PICO_API int pico_group_rms_norm(const float* x, int x_stride, int group_stride,
 #define GN_LAUNCH(TA, W)                                                                                                 \
     pico_launch((group_rms_norm_kernel<TA, W>), grid, block, 0, stream, x, x_stride, group_stride, groups, n, w, eps,     \
                 den_floor, skip, skip_stride, skip_w, skip_head, (const TA*)pre_gate, pre_stride, (const TA*)post_gate,  \
-                post_stride, (TA*)y)
+                post_stride, post_act, (TA*)y)
     if (dtype == PICO_F32) { if (wide) GN_LAUNCH(float, true); else GN_LAUNCH(float, false); }
     else if (dtype == PICO_BF16) { if (wide) GN_LAUNCH(bf16, true); else GN_LAUNCH(bf16, false); }
     else

@@ -15,6 +15,7 @@
 //   RESIDUAL  x_res[m, n] += sum, float32 in place                          (o_proj, down_proj)
 //   SWIGLU    a[m, i] = silu(gate_i) * up_i; rows i (gate) and I + i (up)   (gate_up, no 2I buffer)
 //   CAPPED    the same rows, a[m, i] = g sigmoid(1.702 g) (u + 1) with g = min(gate_i, L), u = clamp(up_i, -L, L)
+//   GELU      the same rows, a[m, i] = gelu_tanh(gate_i + b_i) * (up_i + b_(I + i)), biases optional
 //   ROPE      q/k heads: rows d and d + hd/2 of a head: bias, rotation by the token's position,
 //             q to the query buffer, k and v straight into their cache pages   (qkv projection)
 //   ARGMAX    token[m] = the first n with the largest sum: every block keeps the best of its own tiles, the
@@ -51,8 +52,8 @@
 #define SG_CTAS_PER_SM 2
 #endif
 
-enum { SG_STORE = 0, SG_RESIDUAL = 1, SG_SWIGLU = 2, SG_ROPE = 3, SG_ARGMAX = 4, SG_CAPPED = 5 };
-__host__ __device__ constexpr bool sg_is_glu(int epi) { return epi == SG_SWIGLU || epi == SG_CAPPED; }
+enum { SG_STORE = 0, SG_RESIDUAL = 1, SG_SWIGLU = 2, SG_ROPE = 3, SG_ARGMAX = 4, SG_CAPPED = 5, SG_GELU = 6 };
+__host__ __device__ constexpr bool sg_is_glu(int epi) { return epi == SG_SWIGLU || epi == SG_CAPPED || epi == SG_GELU; }
 
 // ARGMAX: what each block found, and how many blocks have reported (reset by the block that reports last, so
 // launches on one stream need no clearing in between; launches that overlap on the GPU would mix their entries)
@@ -76,10 +77,10 @@ struct SkinnyArgs {
     void* out;                // [M, ld_out] bf16 or float32
     int ld_out;
     int out_f32;
-    const float* bias;        // [N] or null (STORE and ROPE)
+    const float* bias;        // [N] or null (STORE, ROPE and GELU)
     // RESIDUAL
     float* resid;             // [M, N]
-    // SWIGLU, CAPPED: N = 2 * I; out = [M, I] bf16 in `out`
+    // SWIGLU, CAPPED, GELU: N = 2 * I; out = [M, I] bf16 in `out`
     float limit;              // CAPPED: L of g' sigmoid(1.702 g') (u' + 1), g' = min(g, L), u' = clamp(u, -L, L)
     // ROPE
     int nh, nkv, hd, rot_half, page_size;
@@ -188,6 +189,9 @@ __device__ __forceinline__ void sg_epilogue(const SkinnyArgs& p, const float* re
             if (EPI == SG_CAPPED) {
                 const float gc = fminf(gte, p.limit), uc = fminf(fmaxf(up, -p.limit), p.limit);
                 y = gc / (1.0f + expf(-1.702f * gc)) * (uc + 1.0f);
+            } else if (EPI == SG_GELU) {      // g / 2 (1 + tanh(z)) = g / (1 + e^(-2 z)), z = sqrt(2 / pi) (g + 0.044715 g^3)
+                const float gb = gte + (p.bias ? p.bias[row_a + f] : 0.f), ub = up + (p.bias ? p.bias[row_b + f] : 0.f);
+                y = gb / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * gb * gb, gb, gb))) * ub;
             } else {
                 y = gte / (1.0f + expf(-gte)) * up;
             }
@@ -575,6 +579,17 @@ PICO_API int pico_skinny_gate_up_swiglu(const void* x, int ldx, const void* w, v
     a.w = (const bf16*)w; sg_set_x(a, x, ldx, norm_w, eps, nullptr); a.M = M; a.N = 2 * I; a.K = K;
     a.out = out; a.ld_out = I; a.limit = limit;
     return limit > 0.f ? sg_launch<SG_CAPPED>(a, I / 8, stream) : sg_launch<SG_SWIGLU>(a, I / 8, stream);
+}
+
+// out[M, I] = gelu_tanh(x wg^T + bg) * (x wu^T + bu) with w = [wg; wu] of shape [2I, K] and bias = [bg; bu] float32 [2I] or
+// nullptr.  I % 8 == 0.
+PICO_API int pico_skinny_gate_up_gelu(const void* x, int ldx, const void* w, const float* bias, void* out, int M, int I, int K,
+                                      cudaStream_t stream) {
+    if (sg_check(M, 2 * I, K, ldx) || I % 8 != 0) return PICO_ERR_SIZE;
+    SkinnyArgs a = {};
+    a.w = (const bf16*)w; sg_set_x(a, x, ldx, nullptr, 0.f, nullptr); a.M = M; a.N = 2 * I; a.K = K;
+    a.out = out; a.ld_out = I; a.bias = bias;
+    return sg_launch<SG_GELU>(a, I / 8, stream);
 }
 
 // qkv projection with bias, rotary encoding and cache store fused: q_out [M, nh*hd] gets the rotated

@@ -5,6 +5,7 @@ from .zikupel import build_zikupel
 from .zazilix import build_zazilix
 from .banazen import build_banazen
 from .vanapel import build_vanapel
+from .zegorax import build_zegorax
 
 __all__ = ["DecoderModel", "LayerCall", "Binding", "build_qwen2", "build_zapipel", "build_zikupel", "build_zazilix", "build_banazen",
-           "build_vanapel"]
+           "build_vanapel", "build_zegorax"]

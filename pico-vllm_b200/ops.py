@@ -73,7 +73,12 @@ def library():
         "pico_paged_prefill_tcgen05": [vp, vp, vp, i32, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32,
                                        vp, i32, vp, i32, f32, vp, i32, vp, vp, vp],
         "pico_tca_status": [vp],
-        "pico_gemm_tcgen05_pair": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp],
+        "pico_gemm_tcgen05_pair": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, vp],
+        "pico_skinny_gate_up_gelu": [vp, i32, vp, vp, vp, i32, i32, i32, vp],
+        "pico_bias_glu": [vp, vp, i32, vp, i32, i32, i32, vp],
+        "pico_tanh_norm": [vp, vp, f32, vp, f32, vp, f32, vp, vp, vp, vp, vp, i32, i32, i32, vp],
+        "pico_map_rope_store": [vp, i32, i32, i32, i32, vp, vp, i32, f32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp],
+        "pico_map_difference": [vp, vp, i32, f32, f32, f32, vp, i32, i32, i32, i32, i32, vp],
         "pico_tp_status": [vp],
         "pico_sample": [vp, i32, i32, i32, vp, vp, vp, vp, vp],
         "pico_post_add_norm": [vp, vp, vp, i32, f32, vp, i32, f32, vp, vp, i32, i32, i32, i32, i32, vp],
@@ -108,9 +113,9 @@ def library():
         "pico_hgrn2_prepare": [vp, i32, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32, vp],
         "pico_causal_conv_silu": [vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
         "pico_mamba2_prepare": [vp, i32, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, vp],
-        "pico_group_rms_norm": [vp, i32, i32, i32, i32, vp, f32, vp, vp, i32, vp, i32, vp, i32, vp, i32, vp, i32, i32, vp],
-        "pico_delta_prepare": [vp, i32, i32, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, f32, f32, i32, vp],
-        "pico_gated_delta_rule": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+        "pico_group_rms_norm": [vp, i32, i32, i32, i32, vp, f32, vp, vp, i32, vp, i32, vp, i32, vp, i32, i32, vp, i32, i32, vp],
+        "pico_delta_prepare": [vp, i32, i32, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, f32, f32, i32, i32, vp],
+        "pico_gated_delta_rule": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp],
         "pico_pair_rope_norm_store": [vp, i32, i32, i32, i32, vp, vp, i32, i32, vp, vp, f32, vp, vp, vp, vp, i32, i32, i32, i32,
                                       i32, i32, i32, i32, vp],
         "pico_sum_add_norm": [vp, vp, vp, i32, f32, f32, vp, vp, i32, f32, f32, vp, vp, i32, f32, f32, vp, i32, f32, vp, vp, i32,
@@ -680,11 +685,11 @@ def tc_status() -> int:
 TC_PAIR_MIN_TOKENS = 200      # from here on the tcgen05 path pays
 
 
-def _tc_gemm(x, weight, out, residual, M, N, K, epi, rows, what, limit=0.0):
+def _tc_gemm(x, weight, out, residual, M, N, K, epi, rows, what, limit=0.0, bias=None):
     """The tcgen05 product kernel: a tile per pair of blocks (``tcgen05.mma.cta_group::2``).  ``rows``: None = the
     kernel picks its tile; 256 or 512 = that many rows of x per pair."""
     _check(library().pico_gemm_tcgen05_pair(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), _ptr(residual), M, N, K,
-                                            epi, int(rows or 0), float(limit), _stream()), "gemm_tcgen05_pair" + what)
+                                            epi, int(rows or 0), float(limit), _ptr(bias), _stream()), "gemm_tcgen05_pair" + what)
     _count()
 
 
@@ -722,6 +727,75 @@ def tc_gate_up_swiglu(x: torch.Tensor, gate_up_weight: torch.Tensor, rows=None, 
     out = torch.empty((M, I), dtype=torch.bfloat16, device=x.device)
     _tc_gemm(x, gate_up_weight, out, None, M, 2 * I, K, 3 if limit else 2, rows, " (gate_up)", limit or 0.0)
     return out
+
+
+def _glu_bias(bias: Optional[torch.Tensor], rows: int, what: str) -> Optional[torch.Tensor]:
+    _cuda(bias)
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (rows,) or not bias.is_contiguous()):
+        raise KernelError(f"{what}: the biases must be contiguous float32, gate's and then up's")
+    return bias
+
+
+def skinny_gate_up_gelu(x: torch.Tensor, gate_up_weight: torch.Tensor, bias: Optional[torch.Tensor]) -> torch.Tensor:
+    """gelu_tanh(x wg^T + bg) * (x wu^T + bu) for gate_up_weight = [wg; wu] ([2I, K]) and bias = [bg; bu] float32 or None;
+    returns [M, I] bfloat16.  Up to 16 tokens."""
+    _cuda(x, gate_up_weight)
+    if not skinny_takes(x, gate_up_weight):
+        raise KernelError("skinny_gate_up_gelu: needs bfloat16, at most 16 tokens, K and 2I multiples of 16")
+    M, K = x.shape
+    I = gate_up_weight.shape[0] // 2
+    _glu_bias(bias, 2 * I, "skinny_gate_up_gelu")
+    out = torch.empty((M, I), dtype=torch.bfloat16, device=x.device)
+    _check(library().pico_skinny_gate_up_gelu(_ptr(x), x.stride(0), _ptr(gate_up_weight), _ptr(bias), _ptr(out), M, I, K, _stream()),
+           "skinny_gate_up_gelu")
+    _count()
+    return out
+
+
+def tc_gate_up_gelu(x: torch.Tensor, gate_up_weight: torch.Tensor, bias: Optional[torch.Tensor], rows=None) -> torch.Tensor:
+    """As :func:`skinny_gate_up_gelu` for many tokens, on the tcgen05 tensor cores."""
+    _cuda(x, gate_up_weight)
+    if not tc_takes(x, gate_up_weight):
+        raise KernelError("tc_gate_up_gelu: sizes not taken")
+    M, K = x.shape
+    I = gate_up_weight.shape[0] // 2
+    _glu_bias(bias, 2 * I, "tc_gate_up_gelu")
+    out = torch.empty((M, I), dtype=torch.bfloat16, device=x.device)
+    _tc_gemm(x, gate_up_weight, out, None, M, 2 * I, K, 4, rows, " (gate_up, gelu)", bias=bias)
+    return out
+
+
+GLU_ACTS = {"silu": 0, "gelu_tanh": 1}
+
+
+def bias_glu(gate_up: torch.Tensor, bias: Optional[torch.Tensor], act: str) -> torch.Tensor:
+    """act(gate_up[:, :I] + bias[:I]) * (gate_up[:, I:] + bias[I:]), float32 inside; ``act`` "silu" or "gelu_tanh" (a / 2 * (1 +
+    tanh(sqrt(2 / pi) (a + 0.044715 a^3)))); ``bias`` float32 [2I] or None.  Returns [T, I] in gate_up's type."""
+    _cuda(gate_up)
+    T, I = gate_up.shape[0], gate_up.shape[1] // 2
+    if gate_up.dim() != 2 or gate_up.shape[1] != 2 * I or not gate_up.is_contiguous() or act not in GLU_ACTS:
+        raise KernelError("bias_glu: gate_up must be contiguous [T, 2 * I], the activation silu or gelu_tanh")
+    _glu_bias(bias, 2 * I, "bias_glu")
+    out = torch.empty((T, I), dtype=gate_up.dtype, device=gate_up.device)
+    _check(library().pico_bias_glu(_ptr(gate_up), _ptr(bias), GLU_ACTS[act], _ptr(out), T, I, _dtype_code(gate_up), _stream()), "bias_glu")
+    _count()
+    return out
+
+
+def linear_bias(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, bias_act: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x [T, K] times weight[N, K] transposed plus ``bias`` float32 [N].  Up to 16 tokens: this package's product with the bias
+    in its epilogue; more: the library's, whose epilogue takes the bias in the activation type (``bias_act``, made here when it
+    is not given; exact for a bias that was stored in that type)."""
+    _cuda(x, weight, bias)
+    if bias.dtype != torch.float32 or bias.shape != (weight.shape[0],):
+        raise KernelError("linear_bias: the bias must be float32 [N]")
+    if skinny_takes(x, weight):
+        return skinny_linear(x, weight, bias)
+    if x.dtype == weight.dtype:
+        return torch.addmm(bias.to(x.dtype) if bias_act is None else bias_act, x, weight.t())
+    if weight.dtype == torch.float32 and x.dtype == torch.bfloat16:
+        return torch.addmm(bias, x.float(), weight.t()).to(torch.bfloat16)
+    raise KernelError(f"linear_bias: activations {x.dtype} with weights {weight.dtype} is not supported")
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -1439,13 +1513,13 @@ def mamba2_prepare(proj: torch.Tensor, dt_off: int, dt_bias: Optional[torch.Tens
 def group_rms_norm(x: torch.Tensor, groups: int, n: int, group_stride: int, weight: Optional[torch.Tensor], eps: float,
                    out_dtype: torch.dtype, den_floor: Optional[torch.Tensor] = None, skip: Optional[torch.Tensor] = None,
                    skip_w: Optional[torch.Tensor] = None, skip_head: int = 1, pre_gate: Optional[torch.Tensor] = None,
-                   post_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   post_gate: Optional[torch.Tensor] = None, post_act: str = "sigmoid") -> torch.Tensor:
     """The norm that finishes a recurrent mixer, a root mean square per group of ``n`` columns (group g starts at column
     g * group_stride of x, float32 rows).  For column j of group g, col = g * n + j, in this order:
       ``den_floor`` [T, groups]: val /= max(|x[t, g * group_stride + n]|, den_floor[t, g]) + 1e-6 (a normaliser that rides
       as column n of its group);  ``skip`` (float32 rows) with ``skip_w``: val += skip_w[col // skip_head] * skip[t, col];
       ``pre_gate``: val *= silu(pre_gate[t, col]);  y = val / sqrt(mean_j val^2 + eps) * weight[col];
-      ``post_gate``: y *= sigmoid(post_gate[t, col]).  Gates are in ``out_dtype`` (column slices are fine).
+      ``post_gate``: y *= f(post_gate[t, col]), f the function ``post_act`` names ("sigmoid" or "silu").  Gates are in ``out_dtype`` (column slices are fine).
     Returns [T, groups * n] in ``out_dtype``."""
     _cuda(x, weight, den_floor, skip, skip_w, pre_gate, post_gate)
     _f32_rows(x, "group_rms_norm: x")
@@ -1463,11 +1537,14 @@ def group_rms_norm(x: torch.Tensor, groups: int, n: int, group_stride: int, weig
     for g in (pre_gate, post_gate):
         if g is not None and (g.dtype != out_dtype or g.dim() != 2 or g.stride(1) != 1 or g.shape[0] != T or g.shape[1] < N):
             raise KernelError("group_rms_norm: gates must be rows in the output type")
+    if post_act not in ("sigmoid", "silu"):
+        raise KernelError(f"group_rms_norm: post_act {post_act!r} is not built (sigmoid, silu)")
     y = torch.empty((T, N), dtype=out_dtype, device=x.device)
     _check(library().pico_group_rms_norm(_ptr(x), x.stride(0), group_stride, groups, n, _ptr(weight), float(eps), _ptr(den_floor),
                                          _ptr(skip), skip.stride(0) if skip is not None else 0, _ptr(skip_w), int(skip_head),
                                          _ptr(pre_gate), pre_gate.stride(0) if pre_gate is not None else 0, _ptr(post_gate),
-                                         post_gate.stride(0) if post_gate is not None else 0, _ptr(y), T, _dtype_code(y), _stream()),
+                                         post_gate.stride(0) if post_gate is not None else 0, 1 if post_act == "silu" else 0, _ptr(y),
+                                         T, _dtype_code(y), _stream()),
            "group_rms_norm")
     _count()
     return y
@@ -1504,41 +1581,43 @@ def whole_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w
 # ------------------------------------------------------------------------------------------ the delta rule; neighbours that turn together
 def delta_prepare(xc: torch.Tensor, q_off: int, k_off: int, proj: torch.Tensor, b_off: int, dt: torch.Tensor,
                   dt_bias: Optional[torch.Tensor], a_log: torch.Tensor, heads: int, kv_heads: int, dim: int,
-                  unit_eps: float = 1e-6) -> torch.Tensor:
+                  unit_eps: float = 1e-6, per_head: bool = False) -> torch.Tensor:
     """The float32 inputs of the gated delta rule.  ``xc`` float32 rows hold ``kv_heads`` query heads at q_off and as many key
     heads at k_off (``dim`` each); ``proj`` (activation type) one logit per head at b_off; ``dt`` [T, heads * dim] (activation
     type) the decay's argument, ``dt_bias`` float32 [heads * dim], ``a_log`` float32 [heads].  Returns float32 [T, P],
     P = 2 G d + H d + H + G:  q / sqrt(|q|^2 + unit_eps) * d^-1/2  |  k / sqrt(|k|^2 + unit_eps)  |
-    exp(-exp(a_log) softplus(dt + dt_bias))  |  sigmoid(logit)  |  k . q."""
+    exp(-exp(a_log) softplus(dt + dt_bias))  |  sigmoid(logit)  |  k . q.  ``per_head``: one decay a head instead of one a row
+    of its memory (``dt`` [T, heads], ``dt_bias`` [heads]; P = 2 G d + H + H + G)."""
     _cuda(xc, proj, dt, dt_bias, a_log)
     T = xc.shape[0]
     _f32_rows(xc, "delta_prepare: xc")
     H, G, d = heads, kv_heads, dim
+    NA = H if per_head else H * d
     if H % G or max(q_off, k_off) + G * d > xc.shape[1] or proj.dim() != 2 or proj.stride(1) != 1 or b_off + H > proj.shape[1] \
-            or dt.dim() != 2 or dt.stride(1) != 1 or dt.shape != (T, H * d) or dt.dtype != proj.dtype or proj.shape[0] != T:
+            or dt.dim() != 2 or dt.stride(1) != 1 or dt.shape != (T, NA) or dt.dtype != proj.dtype or proj.shape[0] != T:
         raise KernelError("delta_prepare: a row is narrower than its heads")
-    if a_log.dtype != torch.float32 or a_log.shape != (H,) or (dt_bias is not None and (dt_bias.dtype != torch.float32 or dt_bias.shape != (H * d,))):
-        raise KernelError("delta_prepare: a_log float32 [heads], dt_bias float32 [heads * dim]")
-    prep = torch.empty((T, 2 * G * d + H * d + H + G), dtype=torch.float32, device=xc.device)
+    if a_log.dtype != torch.float32 or a_log.shape != (H,) or (dt_bias is not None and (dt_bias.dtype != torch.float32 or dt_bias.shape != (NA,))):
+        raise KernelError("delta_prepare: a_log float32 [heads], dt_bias float32, one per decay")
+    prep = torch.empty((T, 2 * G * d + NA + H + G), dtype=torch.float32, device=xc.device)
     _check(library().pico_delta_prepare(_ptr(xc), xc.stride(0), q_off, k_off, _ptr(proj), proj.stride(0), b_off, _ptr(dt),
                                         dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(prep), T, H, G, d, float(d) ** -0.5,
-                                        float(unit_eps), _dtype_code(proj), _stream()), "delta_prepare")
+                                        float(unit_eps), 1 if per_head else 0, _dtype_code(proj), _stream()), "delta_prepare")
     _count()
     return prep
 
 
 def gated_delta_rule(prep: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seg_slots: torch.Tensor, cu_q: torch.Tensor,
-                     positions: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+                     positions: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, per_head: bool = False) -> torch.Tensor:
     """Per head h, token by token in the order of each segment, from and into ``state`` float32 [slots, heads, vdim, dim] (S
     transposed; row ``seg_slots[s]``):  S <- diag(a) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.  ``prep``: the rows
-    :func:`delta_prepare` made (head h reads query and key head h // (heads / kv_heads)); ``v`` float32 rows with head h's values
+    :func:`delta_prepare` made with the same ``per_head`` (head h reads query and key head h // (heads / kv_heads)); ``v`` float32 rows with head h's values
     at h * vdim (a column slice is fine).  A segment whose first position is negative is padding.  Returns o float32
     [T, heads * vdim]."""
     _cuda(prep, v, state, seg_slots, cu_q, positions)
     _f32_rows(v, "gated_delta_rule: v")
     T, S = prep.shape[0], seg_slots.shape[0]
     H, G, d = heads, kv_heads, dim
-    if prep.dtype != torch.float32 or not prep.is_contiguous() or prep.shape[1] != 2 * G * d + H * d + H + G or v.shape[0] != T \
+    if prep.dtype != torch.float32 or not prep.is_contiguous() or prep.shape[1] != 2 * G * d + (H if per_head else H * d) + H + G or v.shape[0] != T \
             or v.shape[1] < H * vdim:
         raise KernelError("gated_delta_rule: prep must be what delta_prepare returns and v hold every head's values")
     if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (H, vdim, d):
@@ -1552,7 +1631,7 @@ def gated_delta_rule(prep: torch.Tensor, v: torch.Tensor, state: torch.Tensor, s
         raise KernelError("gated_delta_rule: cu_q must have one more entry than seg_slots, positions one per token")
     out = torch.empty((T, H * vdim), dtype=torch.float32, device=prep.device)
     _check(library().pico_gated_delta_rule(_ptr(prep), _ptr(v), v.stride(0), _ptr(state), _ptr(seg_slots), _ptr(cu_q),
-                                           _ptr(positions), _ptr(out), out.stride(0), S, H, G, d, vdim, _stream()),
+                                           _ptr(positions), _ptr(out), out.stride(0), S, H, G, d, vdim, 1 if per_head else 0, _stream()),
            f"gated_delta_rule (dim {d})")
     _count()
     return out
@@ -1660,3 +1739,88 @@ def capped_glu(gu: torch.Tensor, ff: int, limit: float, row_gate_col: Optional[i
            "capped_glu")
     _count()
     return out
+
+
+# ------------------------------------------------------------------------------------------ a squashing instead of a norm
+def tanh_norm(x: torch.Tensor, terms, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: Optional[torch.Tensor],
+              rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """x float32 [T, H] += sum over ``terms`` (up to three) of scale * delta, each a tuple (delta [T, H] in the activation type,
+    scale); then out = tanh(alpha * x) * weight + bias (``alpha`` one float32 number on the device, weight and bias float32 [H];
+    ``out`` None: the adds alone).  With ``rows`` (int32 [R]) out[r] is made from row rows[r] and x is left alone."""
+    terms = list(terms)
+    if len(terms) > 3:
+        raise KernelError("tanh_norm: at most three terms")
+    _cuda(x, alpha, weight, bias, out, rows, *(d for d, _ in terms))
+    H = x.shape[1]
+    R = rows.shape[0] if rows is not None else x.shape[0]
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous():
+        raise KernelError("tanh_norm: x must be contiguous float32 [T, H]")
+    like = out if out is not None else (terms[0][0] if terms else None)
+    if like is None:
+        return None
+    flat = []
+    for d, sc in terms:
+        if d.shape != x.shape or d.dtype != like.dtype or not d.is_contiguous():
+            raise KernelError("tanh_norm: every term must be contiguous, shaped like x, in the activation type")
+        flat += [_ptr(d), float(sc)]
+    flat += [None, 0.0] * (3 - len(terms))
+    if out is not None and (out.shape != (R, H) or not out.is_contiguous()):
+        raise KernelError("tanh_norm: out must be contiguous [rows, H]")
+    if alpha.dtype != torch.float32 or alpha.numel() != 1 or weight.dtype != torch.float32 or bias.dtype != torch.float32 \
+            or weight.shape != (H,) or bias.shape != (H,):
+        raise KernelError("tanh_norm: alpha is one float32 number, weight and bias float32 [H]")
+    if rows is not None and rows.dtype != torch.int32:
+        raise KernelError("tanh_norm: rows must be int32")
+    _check(library().pico_tanh_norm(_ptr(x), *flat, _ptr(alpha), _ptr(weight), _ptr(bias), _ptr(out), _ptr(rows), R, H, _dtype_code(like),
+                                    _stream()), f"tanh_norm (width {H})")
+    _count()
+    return out
+
+
+# ------------------------------------------------------------------------------------------ attention with several maps a head
+def map_rope_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, positions: torch.Tensor, inv_freq: torch.Tensor,
+                   mult: float, slots: Optional[torch.Tensor], k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor],
+                   heads: int, kv_heads: int, maps: int, dim: int, vdim: int, row: int, page_size: int) -> torch.Tensor:
+    """Per token row [q: heads x maps x dim | k: kv_heads x maps x dim | v: kv_heads x vdim] (at the given offsets): the first
+    2 * len(inv_freq) numbers of every query and key map turn (i with i + len(inv_freq), by position * inv_freq[i], cos and sin
+    times ``mult``); a key head's maps go side by side into its key row, the values into theirs (``slots`` int32: page *
+    page_size + offset, -1 or None: not stored; pages [pages, kv_heads, page_size, row], zero-padded).  Returns the queries
+    [T, heads * maps * row]: query map m of a head is a row of zeros with the map in the place of key map m."""
+    _cuda(proj, positions, inv_freq, slots, k_pages, v_pages)
+    T = proj.shape[0]
+    if proj.dim() != 2 or proj.stride(1) != 1 or row < max(maps * dim, vdim) \
+            or max(q_off + heads * maps * dim, k_off + kv_heads * maps * dim, v_off + kv_heads * vdim) > proj.shape[1]:
+        raise KernelError("map_rope_store: the projection row is narrower than its parts, or a head wider than its row")
+    if positions.dtype != torch.int32 or positions.shape != (T,) or inv_freq.dtype != torch.float32 or 2 * inv_freq.shape[0] > dim:
+        raise KernelError("map_rope_store: positions int32 [T], inv_freq float32 [<= dim / 2]")
+    if slots is not None:
+        if slots.dtype != torch.int32 or slots.shape != (T,) or k_pages is None or v_pages is None:
+            raise KernelError("map_rope_store: slots must be int32 [T] and come with pages")
+        for pg in (k_pages, v_pages):
+            if pg.dtype != proj.dtype or not pg.is_contiguous() or tuple(pg.shape[1:]) != (kv_heads, page_size, row):
+                raise KernelError("map_rope_store: pages must be contiguous [pages, kv_heads, page_size, row] in proj's type")
+    q = torch.empty((T, heads * maps * row), dtype=proj.dtype, device=proj.device)
+    _check(library().pico_map_rope_store(_ptr(proj), proj.stride(0), q_off, k_off, v_off, _ptr(positions), _ptr(inv_freq),
+                                         inv_freq.shape[0], float(mult), _ptr(slots), _ptr(k_pages), _ptr(v_pages), _ptr(q), T, heads,
+                                         kv_heads, maps, dim, vdim, row, page_size, _dtype_code(proj), _stream()), "map_rope_store")
+    _count()
+    return q
+
+
+def map_difference(a: torch.Tensor, heads: int, row: int, vdim: int, lam: float, eps: float, factor: float,
+                   gate_logits: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """From a [T, heads, 2, row] (flat rows; the first ``vdim`` numbers of each count): o = a_1 - lam * a_2, then o / sqrt(mean(o^2)
+    + eps) * factor, times sigmoid(gate_logits[t, head]) when given (rows in a's type, a column slice is fine).  Returns
+    [T, heads * vdim] in a's type."""
+    _cuda(a, gate_logits)
+    T = a.shape[0]
+    if a.dim() != 2 or not a.is_contiguous() or a.shape[1] != heads * 2 * row or row < vdim:
+        raise KernelError("map_difference: a must be contiguous [T, heads * 2 * row]")
+    if gate_logits is not None and (gate_logits.dtype != a.dtype or gate_logits.shape != (T, heads) or gate_logits.stride(1) != 1):
+        raise KernelError("map_difference: gate logits [T, heads] in a's type with contiguous rows")
+    y = torch.empty((T, heads * vdim), dtype=a.dtype, device=a.device)
+    _check(library().pico_map_difference(_ptr(a), _ptr(gate_logits), gate_logits.stride(0) if gate_logits is not None else 0, float(lam),
+                                         float(eps), float(factor), _ptr(y), T, heads, row, vdim, _dtype_code(a), _stream()),
+           "map_difference")
+    _count()
+    return y

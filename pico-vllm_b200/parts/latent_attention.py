@@ -10,11 +10,16 @@ cached latent rank r:
 
 No position encoding acts on q or k.  A layer may read the latents another layer caches (``own_latent=False``: it
 has no W_dkv; its cache entry is that layer's).  Options: ``q_rank=None`` - the queries are projected directly, q = W_q h
-(no query latent, no norm on that side); ``gate=False`` - no output gate; ``window`` W - position i sees the last W
+(no query latent, no norm on that side); ``gate=False`` - no output gate; ``gate="elements"`` - the gate has a logit for every
+number of the concatenated heads (W_g has H d_v rows) instead of one per head; ``window`` W - position i sees the last W
 positions, itself included; ``rot_dim`` with ``position`` - beside the unrotated d numbers a head has rot_dim rotated ones, and
 W_dkv makes rot_dim more numbers, one rotated key part k_r shared by all heads and not normed:
 
     q_a = [ u_a (d) | rot(r_a) (rot_dim) ],  p_a(j) = softmax_j( scale * (u_a . k_a(j) + rot(r_a) . rot(k_r(j))) )
+
+A position encoding with ``pairing`` "neighbours" turns dimensions 2i and 2i + 1 together: the rows of W_uq and W_dkv that make the
+rotated part are put in the order 0, 2, 4, ..., 1, 3, 5, ... when they are loaded, the same order on both sides, which leaves
+every score as it is and turns the pairs into (i, i + n/2), the ones the kernels have.
 
 ``sink`` - the softmax's denominator has one more term exp(sink_a), a learned number per head.
 
@@ -31,7 +36,7 @@ W_o product.  Norms, gate and softmax are float32.
 """
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import List, Optional, Union
 
 import torch
 
@@ -56,13 +61,17 @@ def _linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 @register("mixer", "latent_attention")
 class LatentAttention(Part):
     def __init__(self, width: int, heads: int, dim: int, vdim: int, q_rank: Optional[int], kv_rank: int, scale: float, eps: float,
-                 own_latent: bool = True, window: Optional[int] = None, gate: bool = True, cache_window="same",
+                 own_latent: bool = True, window: Optional[int] = None, gate: Union[bool, str] = True, cache_window="same",
                  rot_dim: int = 0, position: Optional[Part] = None, sink: bool = False):
         """``cache_window``: how many of the last latents the cache has to keep (None: all); by default the mixer's own
         window.  Layers that read one cache entry through different windows all name the longest."""
         self.width, self.heads, self.dim, self.vdim = width, heads, dim, vdim
         self.q_rank, self.kv_rank, self.scale, self.eps = q_rank, kv_rank, float(scale), float(eps)
-        self.own_latent, self.window, self.gate = own_latent, window, gate
+        if gate not in (True, False, "elements"):
+            raise ConfigError(f"latent_attention: gate {gate!r} must be True (one per head), False or 'elements'")
+        self.own_latent, self.window = own_latent, window
+        self.gate_rows = heads * vdim if gate == "elements" else heads if gate else 0
+        self.gate_elements = gate == "elements"
         self.cache_window = window if cache_window == "same" else cache_window
         if (rot_dim > 0) != (position is not None) or getattr(position, "rot_dim", 0) > rot_dim:
             raise ConfigError("latent_attention: a rotated part needs a position encoding of at most its size")
@@ -75,8 +84,8 @@ class LatentAttention(Part):
         down = [Piece("dq.weight", (self.q_rank, self.width))] if self.q_rank else []
         if self.own_latent:
             down.append(Piece("dkv.weight", (self.kv_rank + self.rot_dim, self.width)))
-        if self.gate:
-            down.append(Piece("g.weight", (self.heads, self.width)))
+        if self.gate_rows:
+            down.append(Piece("g.weight", (self.gate_rows, self.width)))
         ps = [Param("down_weight", tuple(down))] if down else []
         if self.q_rank:
             ps += [Param("q_norm", (Piece("dq.norm", (self.q_rank,)),), kind="vector", init="one_plus_normal"),
@@ -97,6 +106,15 @@ class LatentAttention(Part):
         [H, d, row] and W_uv transposed as [H, row, d_v], both with zeros beyond kv_rank.  A rotated part adds rot_dim rows to
         W_uk that hand the query's rotated numbers on to their places behind the latent."""
         pad = self.row - self.kv_rank
+        if self.rot_dim and getattr(self.position, "pairing", "rot_half") == "neighbours":
+            n = self.position.rot_dim
+            order = list(range(0, n, 2)) + list(range(1, n, 2)) + list(range(n, self.rot_dim))
+            if attr == "down_weight" and self.own_latent:
+                at = (self.q_rank or 0) + self.kv_rank
+                tensor = torch.cat([tensor[:at], tensor[at:at + self.rot_dim][order], tensor[at + self.rot_dim:]], 0)
+            elif attr == "uq_weight":
+                t = tensor.view(self.heads, self.dim + self.rot_dim, -1)
+                tensor = torch.cat([t[:, :self.dim], t[:, self.dim:][:, order]], 1).reshape(tensor.shape)
         if attr == "down_weight":
             extra = _round_up(tensor.shape[0], 16) - tensor.shape[0]
             if extra:
@@ -138,7 +156,7 @@ class LatentAttention(Part):
         latent = cache.tensors["latent"]                       # [pages, 1, page_size, R]
         stores = self.own_latent and cache.store
         q_rank = self.q_rank or 0
-        cq, gate = h, None
+        cq, gate, elements = h, None, None
         if self.down_weight is not None:
             proj = _linear(h, self.down_weight)
             kv_off = q_rank
@@ -148,7 +166,10 @@ class LatentAttention(Part):
                 rot = (kv_off + self.kv_rank, self.rot_dim, batch.positions, self.position.inv_freq, getattr(self.position, "mult", 1.0))
             cq, gate = ops.latent_norm_store(proj, 0, q_rank, self.q_norm, kv_off, self.kv_rank if stores else 0,
                                              self.kv_norm if stores else None, gb.slots if stores else None,
-                                             latent if stores else None, g_off, H if self.gate else 0, self.eps, rot=rot)
+                                             latent if stores else None, g_off,
+                                             0 if self.gate_elements else self.gate_rows, self.eps, rot=rot)
+            if self.gate_elements:
+                elements = proj[:, g_off:g_off + self.gate_rows]
             if not q_rank:
                 cq = h
         q = _linear(cq, self.uq_weight)                         # [T, H d]: from the query latent, or from h itself
@@ -169,4 +190,6 @@ class LatentAttention(Part):
                                 cache.page_size, self.window, self.scale, splits, batch.scratch, sinks=self.sinks)
         o = torch.empty((T, H * self.vdim), dtype=h.dtype, device=h.device)
         ops.head_linear(oa, self.uv_weight, o, gate)            # o_a = gate_a * W_uv[a] o'_a
+        if elements is not None:
+            ops.sigmoid_gate(o, elements)
         return _linear(o, self.o_weight)

@@ -165,6 +165,34 @@ class CentredNorm(Part):
         return _post_add_norm(self, ops.NORM_CENTRED, x, delta, rows)
 
 
+@register("norm", "tanh_norm")
+class TanhNorm(Part):
+    """y = tanh(alpha * x) * weight + bias: a squashing in the place of a norm, without a mean or a variance; alpha one learned
+    number, weight and bias one per coordinate (Zhu, Chen, He, LeCun, Liu: "Transformers without Normalization").  What is
+    pending is added on the way, up to three outputs at once; outputs that still have to pass a norm of their own are refused."""
+
+    def __init__(self, width: int):
+        self.width = width
+        self.alpha = self.weight = self.bias = None
+        self.act_dtype = torch.bfloat16
+
+    def params(self) -> List[Param]:
+        return [Param("alpha", (Piece("alpha", ()),), kind="vector", init="const:0.5"),
+                Param("weight", (Piece("weight", (self.width,)),), kind="vector", init="one_plus_normal"),
+                Param("bias", (Piece("bias", (self.width,)),), kind="vector")]
+
+    def materialize(self, device, dtype):
+        self.act_dtype = dtype
+
+    def add_norm(self, x: torch.Tensor, delta: Union[None, torch.Tensor, SumDelta],
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if x.dim() != 2 or isinstance(delta, NormedDelta) or (isinstance(delta, SumDelta) and any(n is not None for _, n, _ in delta.terms)):
+            raise KernelError("tanh_norm: built for one residual stream and outputs that need no norm of their own")
+        terms = [] if delta is None else [(d, s) for d, _, s in delta.terms] if isinstance(delta, SumDelta) else [(delta, 1.0)]
+        out = torch.empty((x.shape[0] if rows is None else rows.shape[0], self.width), dtype=self.act_dtype, device=x.device)
+        return ops.tanh_norm(x, terms, self.alpha, self.weight, self.bias, out, rows)
+
+
 @register("norm", "none")
 class PassNorm(Part):
     """No norm at all: ``add_norm`` adds what is pending to the residual stream and hands the stream on in the

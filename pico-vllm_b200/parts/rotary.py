@@ -83,6 +83,44 @@ class YarnRotary(Part):
         self.inv_freq = self.frequencies().to(device)
 
 
+@register("position", "band_scaled_rotary")
+class BandScaledRotary(Part):
+    """Rotary encoding on the first ``rot_dim`` dimensions of a head with frequencies f_i = theta^(-2i/rot_dim) scaled band by
+    band (the rule of Llama 3.1's configuration): with the wavelength l = 2 pi / f,
+
+        l < original / high:  f            l > original / low:  f / factor
+        between:  (1 - s) f / factor + s f,   s = (original / l - low) / (high - low)
+
+    ``factor`` None: plain frequencies.  ``pairing``: "rot_half" (dimension i with i + rot_dim / 2) or "neighbours" (2i with
+    2i + 1; a mixer that cannot turn those may reorder the rows of its projections when they are loaded)."""
+
+    def __init__(self, head_dim: int, theta: float, rot_dim: int = None, factor: float = None, low: float = 1.0, high: float = 4.0,
+                 original: float = 0.0, pairing: str = "rot_half"):
+        self.head_dim, self.theta, self.pairing = head_dim, float(theta), pairing
+        self.rot_dim = head_dim if rot_dim is None else rot_dim
+        if self.rot_dim % 2 or not 0 <= self.rot_dim <= head_dim:
+            raise ConfigError(f"band_scaled_rotary: rot_dim {self.rot_dim} must be even and at most head_dim {head_dim}")
+        if pairing not in ("rot_half", "neighbours"):
+            raise ConfigError(f"band_scaled_rotary: pairing {pairing!r} is not built (rot_half, neighbours)")
+        if factor is not None and (factor <= 0 or original <= 0 or low <= 0 or high < low):
+            raise ConfigError("band_scaled_rotary: factor, original and low must be positive and high at least low")
+        self.factor, self.low, self.high, self.original = factor, low, high, original
+        self.mult = 1.0
+        self.inv_freq = None
+
+    def frequencies(self) -> torch.Tensor:
+        i = torch.arange(self.rot_dim // 2, dtype=torch.float64)
+        f = self.theta ** (-2.0 * i / self.rot_dim) if self.rot_dim else i
+        if self.factor is not None and self.rot_dim:
+            turns = self.original * f / (2.0 * math.pi)          # original / wavelength
+            s = ((turns - self.low) / max(self.high - self.low, 1e-300)).clamp(0.0, 1.0)
+            f = torch.where(turns > self.high, f, torch.where(turns < self.low, f / self.factor, (1.0 - s) * f / self.factor + s * f))
+        return f.to(torch.float32)
+
+    def materialize(self, device, dtype):
+        self.inv_freq = self.frequencies().to(device)
+
+
 @register("position", "none")
 class NoPosition(Part):
     pairing = "half"

@@ -57,6 +57,9 @@ def _register_builtin() -> None:
     from .config.vanapel import VanapelConfig
     from .models.vanapel import build_vanapel
     register_architecture("Vanapel", VanapelConfig, build_vanapel)
+    from .config.zegorax import ZegoraxConfig
+    from .models.zegorax import build_zegorax
+    register_architecture("Zegorax", ZegoraxConfig, build_zegorax)
 
 
 _register_builtin()

@@ -566,7 +566,7 @@ def mamba2_prepare(proj, dt_off, dt_bias, a_log, x, heads, vdim):
 
 
 def group_rms_norm(x, groups, n, group_stride, weight, eps, out_dtype, den_floor=None, skip=None, skip_w=None, skip_head=1,
-                   pre_gate=None, post_gate=None):
+                   pre_gate=None, post_gate=None, post_act="sigmoid"):
     T, N = x.shape[0], groups * n
     val = torch.stack([x[:, g * group_stride:g * group_stride + n] for g in range(groups)], 1)          # [T, groups, n]
     if den_floor is not None:
@@ -582,7 +582,8 @@ def group_rms_norm(x, groups, n, group_stride, weight, eps, out_dtype, den_floor
     if weight is not None:
         y = y * weight
     if post_gate is not None:
-        y = y * torch.sigmoid(post_gate[:, :N].float())
+        z = post_gate[:, :N].float()
+        y = y * torch.sigmoid(z) * (z if post_act == "silu" else 1.0)
     return y.to(out_dtype)
 
 
@@ -616,26 +617,27 @@ NAMES = ["rotate_tail", "head_norm_store", "hyper_expand", "hyper_step", "scale_
          "mma_attention_takes", "paged_attention_mma", "make_kv_tensor_map", "make_kv_tensor_map_2d", "tc_takes", "skinny_takes", "skinny_norm_takes", "skinny_linear", "skinny_linear_residual",
          "skinny_gate_up_swiglu", "skinny_qkv_rope_store",
          "linear", "logits_linear", "sample", "delta_prepare", "gated_delta_rule", "pair_rope_norm_store", "sum_add_norm",
-         "gelu_gate_rows", "capped_glu"]
+         "gelu_gate_rows", "capped_glu", "tanh_norm", "map_rope_store", "map_difference", "bias_glu", "linear_bias", "skinny_gate_up_gelu"]
 
 
-def delta_prepare(xc, q_off, k_off, proj, b_off, dt, dt_bias, a_log, heads, kv_heads, dim, unit_eps=1e-6):
+def delta_prepare(xc, q_off, k_off, proj, b_off, dt, dt_bias, a_log, heads, kv_heads, dim, unit_eps=1e-6, per_head=False):
     T, H, G, d = xc.shape[0], heads, kv_heads, dim
     q = xc[:, q_off:q_off + G * d].reshape(T, G, d)
     k = xc[:, k_off:k_off + G * d].reshape(T, G, d)
     q = q / torch.sqrt((q * q).sum(-1, keepdim=True) + unit_eps) * d ** -0.5
     k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + unit_eps)
     z = dt.float() + (dt_bias if dt_bias is not None else 0.0)
-    keep = torch.exp(-torch.exp(a_log).repeat_interleave(d) * torch.nn.functional.softplus(z, threshold=20.0))
+    keep = torch.exp(-torch.exp(a_log).repeat_interleave(1 if per_head else d) * torch.nn.functional.softplus(z, threshold=20.0))
     beta = torch.sigmoid(proj[:, b_off:b_off + H].float())
     return torch.cat([q.reshape(T, -1), k.reshape(T, -1), keep, beta, (q * k).sum(-1)], 1).contiguous()
 
 
-def gated_delta_rule(prep, v, state, seg_slots, cu_q, positions, heads, kv_heads, dim, vdim):
+def gated_delta_rule(prep, v, state, seg_slots, cu_q, positions, heads, kv_heads, dim, vdim, per_head=False):
     T, H, G, d = prep.shape[0], heads, kv_heads, dim
     q, k = prep[:, :G * d].reshape(T, G, d), prep[:, G * d:2 * G * d].reshape(T, G, d)
-    keep = prep[:, 2 * G * d:2 * G * d + H * d].reshape(T, H, d)
-    beta = prep[:, 2 * G * d + H * d:2 * G * d + H * d + H]
+    NA = H if per_head else H * d
+    keep = prep[:, 2 * G * d:2 * G * d + NA].reshape(T, H, -1)
+    beta = prep[:, 2 * G * d + NA:2 * G * d + NA + H]
     out = torch.zeros(T, H * vdim)
     for s in range(seg_slots.shape[0]):
         a0, a1 = int(cu_q[s]), int(cu_q[s + 1])
@@ -717,6 +719,74 @@ def gelu_gate_rows(z, table, off, tokens, feedback=None):
     a = z.float()
     g = 0.5 * a * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (a + 0.044715 * a ** 3)))
     return (g * table[ids.clamp(min=0), off:off + z.shape[1]].float()).to(z.dtype)
+
+
+# ------------------------------------------------------------------ a squashing norm, several maps a head, biased activations
+def tanh_norm(x, terms, alpha, weight, bias, out, rows=None):
+    src = x if rows is None else x[rows.long()]
+    acc = src.clone()
+    for delta, s in terms:
+        acc = acc + s * (delta if rows is None else delta[rows.long()]).float()
+    if rows is None:
+        x.copy_(acc)
+    if out is not None:
+        out.copy_((torch.tanh(float(alpha) * acc) * weight + bias).to(out.dtype))
+    return out
+
+
+def map_rope_store(proj, q_off, k_off, v_off, positions, inv_freq, mult, slots, k_pages, v_pages, heads, kv_heads, maps, dim, vdim,
+                   row, page_size):
+    T, r = proj.shape[0], inv_freq.shape[0]
+    p = proj.float()
+    ang = positions.float()[:, None] * inv_freq[None, :]
+    c, s = (ang.cos() * mult)[:, None, None, :], (ang.sin() * mult)[:, None, None, :]
+    live = (positions >= 0)[:, None, None, None]
+
+    def turn(t):
+        a, b = t[..., :r], t[..., r:2 * r]
+        return torch.where(live, torch.cat([a * c - b * s, b * c + a * s, t[..., 2 * r:]], -1), t)
+    q = turn(p[:, q_off:q_off + heads * maps * dim].reshape(T, heads, maps, dim))
+    k = turn(p[:, k_off:k_off + kv_heads * maps * dim].reshape(T, kv_heads, maps, dim)).reshape(T, kv_heads, maps * dim)
+    v = p[:, v_off:v_off + kv_heads * vdim].reshape(T, kv_heads, vdim)
+    if slots is not None:
+        for t, sl in enumerate(slots.tolist()):
+            if sl >= 0:
+                for pages, u in ((k_pages, k), (v_pages, v)):
+                    pages[sl // page_size, :, sl % page_size, :] = 0
+                    pages[sl // page_size, :, sl % page_size, :u.shape[2]] = u[t].to(pages.dtype)
+    out = torch.zeros(T, heads, maps, row)
+    for m in range(maps):
+        out[:, :, m, m * dim:(m + 1) * dim] = q[:, :, m]
+    return out.reshape(T, -1).to(proj.dtype)
+
+
+def map_difference(a, heads, row, vdim, lam, eps, factor, gate_logits=None):
+    T = a.shape[0]
+    x = a.float().view(T, heads, 2, row)[..., :vdim]
+    y = _rms_unit(x[:, :, 0] - lam * x[:, :, 1], eps) * factor
+    if gate_logits is not None:
+        y = y * torch.sigmoid(gate_logits.float())[:, :, None]
+    return y.reshape(T, -1).to(a.dtype)
+
+
+def _biased(gu, bias, act):
+    z = gu.float() + (bias if bias is not None else 0.0)
+    I = z.shape[1] // 2
+    g, u = z[:, :I], z[:, I:]
+    f = g * torch.sigmoid(g) if act == "silu" else 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+    return f * u
+
+
+def bias_glu(gate_up, bias, act):
+    return _biased(gate_up, bias, act).to(gate_up.dtype)
+
+
+def skinny_gate_up_gelu(x, gate_up_weight, bias):
+    return _biased(x.float() @ gate_up_weight.float().t(), bias, "gelu_tanh").to(torch.bfloat16)
+
+
+def linear_bias(x, weight, bias, bias_act=None):
+    return (x.float() @ weight.float().t() + bias).to(x.dtype)
 
 
 def install(monkeypatch):
