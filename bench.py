@@ -631,10 +631,30 @@ def vanapel_config(shape, layers):
     return dict(architecture="Vanapel", vocab=DESIGN_VOCAB, width=s["width"], norm=dict(eps=1e-5, groups=2), layers=zl)
 
 
+def zegorax_config(shape, layers):
+    """The Zegorax design at the sizes of ``shape``: of every three layers one has the gated delta rule (as many heads, half as many
+    query/key heads, keys and values of the head size), one differential attention (as many heads on the shape's key/value
+    heads, two maps of half the head size over values of the head size, half of every map rotated with scaled frequencies), one
+    latent attention over a window of 1,024 positions (a quarter of every head rotated; latent and rotated key part together
+    as wide as the shape's latent); the first layer has the dense feed-forward, the others route ``top`` of ``experts`` experts
+    (together as wide as the dense one); no layer runs twice."""
+    s = DESIGN_SHAPES[shape]
+    H, d = s["heads"], s["head"]
+    delta = dict(heads=H, kv_heads=H // 2, dim=d, vdim=d, conv=4)
+    att = dict(heads=H, kv_heads=s["kv_heads"], dim=d // 2, vdim=d, scale=(d // 2) ** -0.5, diff=0.5,
+               rot=dict(base=500000.0, dims=d // 4, scaling=dict(factor=8.0, low=1.0, high=4.0, original=2048)))
+    lat = dict(heads=H, dim=d * 3 // 4, rot_dim=d // 4, vdim=d, q_rank=s["q_rank"], kv_rank=s["kv_rank"] - d // 4, scale=d ** -0.5,
+               rot=dict(base=500000.0, dims=d // 4), mask=dict(size=1024))
+    moe = dict(kind="moe", expert=dict(ff=s["ff"] // s["top"]), router=dict(experts=s["experts"], top=s["top"]))
+    kinds = [("delta", delta), ("attention", att), ("latent_attention", lat)]
+    zl = [dict(type=kinds[i % 3][0], mixer=kinds[i % 3][1], mlp=dict(kind="dense", ff=s["ff"]) if i == 0 else moe) for i in range(layers)]
+    return dict(architecture="Zegorax", vocab=DESIGN_VOCAB, width=s["width"], norm=dict(eps=1e-5), max_positions=8192, layers=zl)
+
+
 # the models a design is measured beside: the closest ones the package had before it (zapipel_dense: the Zapipel design with
 # latents of its own and the dense feed-forward in every layer)
 DESIGN_BESIDE = {"zapipel": ["qwen2"], "zikupel": ["qwen2"], "zazilix": ["zikupel"], "banazen": ["zazilix"],
-                 "vanapel": ["zapipel_dense", "qwen2"]}
+                 "vanapel": ["zapipel_dense", "qwen2"], "zegorax": ["banazen"]}
 
 
 def design_configs(shape, layers):
@@ -656,7 +676,8 @@ def design_configs(shape, layers):
                 num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=s["head"],
                 intermediate_size=s["ff"], tie_word_embeddings=False)
     return {"zapipel": zap, "qwen2": qwen, "zikupel": zikupel_config(shape, layers), "zazilix": zazilix_config(shape, layers),
-            "banazen": banazen_config(shape, layers), "vanapel": vanapel_config(shape, layers), "zapipel_dense": zap_dense}
+            "banazen": banazen_config(shape, layers), "vanapel": vanapel_config(shape, layers), "zegorax": zegorax_config(shape, layers),
+            "zapipel_dense": zap_dense}
 
 
 def run_design(args):
@@ -811,12 +832,12 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 and 64")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one phase only and print a short line (for profiling; not a bench value)")
-    ap.add_argument("--design", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel"], default=None,
+    ap.add_argument("--design", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel", "zegorax"], default=None,
                     help="the named design beside the closest earlier model at equal sizes (zapipel, zikupel: the Qwen2 decoder; "
-                         "zazilix: zikupel; banazen: zazilix; vanapel: zapipel with dense layers, and the Qwen2 decoder), "
+                         "zazilix: zikupel; banazen: zazilix; vanapel: zapipel with dense layers, and the Qwen2 decoder; zegorax: banazen), "
                          "prefill and decode; not the default run")
     ap.add_argument("--shape", choices=sorted(DESIGN_SHAPES) + ["all"], default="all", help="with --design: which sizes")
-    ap.add_argument("--arch", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel", "zapipel_dense", "qwen2", "both"],
+    ap.add_argument("--arch", choices=["zapipel", "zikupel", "zazilix", "banazen", "vanapel", "zegorax", "zapipel_dense", "qwen2", "both"],
                     default="both", help="with --design: which model (both: the design and what it is measured beside)")
     ap.add_argument("--micro", action="store_true",
                     help="time single decode kernels replayed from a graph (skinny products, decode attention)")

@@ -501,7 +501,7 @@ def test_keys_just_inside_and_just_outside_a_window(dtype, window, rank):
     at the window's length and at page borders."""
     raw = _model(97, 64, [_layer(_lat(4, 32, 16, 32, 48, rank, 1.2, window, 10000.0))])
     tensors = _without_positions(_tensors(raw, 91))
-    tensors["l0.mix.o"] = tensors["l0.mix.o"] * 4
+    tensors["l0.mix.o"] = tensors["l0.mix.o"] * 16
     ids = helpers.random_ids(4 * window + 9, raw["vocab"], 6)
     reqs = {"r": ids}
     logits = _oracle(raw, tensors, reqs)
@@ -525,10 +525,13 @@ def test_keys_just_inside_and_just_outside_a_window(dtype, window, rank):
 def test_a_far_key_among_hundreds_and_the_first_tokens(dtype, kind):
     """420 equal tokens but one, at position 3, chosen so that the last queries notice it: losing it would show.  Read from a
     whole prompt, token by token, and in portions."""
-    layer = _lat(2, 48, 16, 32, 32, 48, 1.0) if kind == "latent" else _att(2, 1, 32, 64, 3.0, 0.3, _rot(10000.0, 8, (8.0, 1.0, 4.0, 64)))
+    layer = _lat(2, 48, 16, 32, 32, 48, 1.0) if kind == "latent" else _att(2, 1, 32, 64, 6.0, 0.3, _rot(10000.0, 8, (8.0, 1.0, 4.0, 64)))
     raw = _model(97, 64, [_layer(layer)])
     tensors = _without_positions(_tensors(raw, 17))
-    tensors["l0.mix.o"] = tensors["l0.mix.o"] * 4
+    if kind == "attention":      # equal values cancel in the difference of the maps: one map has to prefer the odd token clearly
+        for n in ("q", "k"):
+            tensors[f"l0.mix.{n}"] = tensors[f"l0.mix.{n}"] * 3
+    tensors["l0.mix.o"] = tensors["l0.mix.o"] * (16 if kind == "attention" else 4)
     base = [11] * 420
     plain_last = plain.forward(raw, tensors, base)[-1]
     best, best_diff = None, 0.0
