@@ -146,12 +146,41 @@ __global__ void sigmoid_gate_kernel(TA* __restrict__ o, const TA* __restrict__ g
     }
 }
 
+// 16 bytes per access: n and g_stride multiples of W = 16 / sizeof(TA), both pointers 16-byte aligned.
+template <typename TA>
+__global__ void sigmoid_gate_vec_kernel(TA* __restrict__ o, const TA* __restrict__ g, int g_stride, int n, int items) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int W = 16 / (int)sizeof(TA);
+    const int idx = blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= items) return;
+    const int per = n / W, t = idx / per, c = (idx - t * per) * W;
+    uint4 raw = *reinterpret_cast<const uint4*>(o + (size_t)idx * W);
+    const uint4 graw = *reinterpret_cast<const uint4*>(g + (size_t)t * g_stride + c);
+    TA* v = reinterpret_cast<TA*>(&raw);
+    const TA* z = reinterpret_cast<const TA*>(&graw);
+#pragma unroll
+    for (int k = 0; k < W; ++k) v[k] = from_f32<TA>(to_f32(v[k]) / (1.0f + expf(-to_f32(z[k]))));
+    *reinterpret_cast<uint4*>(o + (size_t)idx * W) = raw;
+}
+
 PICO_API int pico_sigmoid_gate(void* o, const void* g, int g_stride, int T, int n, int dtype, cudaStream_t stream) {
     if (T <= 0 || n <= 0) return 0;
     const size_t total = (size_t)T * n;
     const long long cap = 16LL * pico_num_sms();
     const size_t want = (total + 255) / 256;
     const int blocks = (int)((long long)want > cap ? cap : (long long)want);
+    const int w = dtype == PICO_F32 ? 4 : 8;
+    if ((dtype == PICO_F32 || dtype == PICO_BF16) && n % w == 0 && g_stride % w == 0 && (((uintptr_t)o | (uintptr_t)g) & 15) == 0 &&
+        total / w <= 0x7fffffffULL) {
+        const int items = (int)(total / w);
+        const dim3 grid((items + 127) / 128);
+        if (dtype == PICO_F32)
+            pico_launch((sigmoid_gate_vec_kernel<float>), grid, dim3(128), 0, stream, (float*)o, (const float*)g, g_stride, n, items);
+        else
+            pico_launch((sigmoid_gate_vec_kernel<bf16>), grid, dim3(128), 0, stream, (bf16*)o, (const bf16*)g, g_stride, n, items);
+        return pico_launch_status();
+    }
     if (dtype == PICO_F32)
         pico_launch((sigmoid_gate_kernel<float>), dim3(blocks), dim3(256), 0, stream, (float*)o, (const float*)g, g_stride, n, total);
     else if (dtype == PICO_BF16)

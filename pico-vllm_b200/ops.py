@@ -114,8 +114,8 @@ def library():
         "pico_causal_conv_silu": [vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
         "pico_mamba2_prepare": [vp, i32, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, vp],
         "pico_group_rms_norm": [vp, i32, i32, i32, i32, vp, f32, vp, vp, i32, vp, i32, vp, i32, vp, i32, i32, vp, i32, i32, vp],
-        "pico_delta_prepare": [vp, i32, i32, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, f32, f32, i32, i32, vp],
-        "pico_gated_delta_rule": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp],
+        "pico_delta_prepare": [vp, i32, i32, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, f32, f32, i32, i32, i32, vp],
+        "pico_gated_delta_rule": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp],
         "pico_pair_rope_norm_store": [vp, i32, i32, i32, i32, vp, vp, i32, i32, vp, vp, f32, vp, vp, vp, vp, i32, i32, i32, i32,
                                       i32, i32, i32, i32, vp],
         "pico_sum_add_norm": [vp, vp, vp, i32, f32, f32, vp, vp, i32, f32, f32, vp, vp, i32, f32, f32, vp, i32, f32, vp, vp, i32,
@@ -1579,15 +1579,20 @@ def whole_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w
 
 
 # ------------------------------------------------------------------------------------------ the delta rule; neighbours that turn together
+DELTA_BLOCK_MIN_TOKENS = 4         # the longest segment of a step from which the delta rule with a decay per head takes four tokens at a time
+
+
 def delta_prepare(xc: torch.Tensor, q_off: int, k_off: int, proj: torch.Tensor, b_off: int, dt: torch.Tensor,
                   dt_bias: Optional[torch.Tensor], a_log: torch.Tensor, heads: int, kv_heads: int, dim: int,
-                  unit_eps: float = 1e-6, per_head: bool = False) -> torch.Tensor:
+                  unit_eps: float = 1e-6, per_head: bool = False, max_q_len: int = 1) -> torch.Tensor:
     """The float32 inputs of the gated delta rule.  ``xc`` float32 rows hold ``kv_heads`` query heads at q_off and as many key
     heads at k_off (``dim`` each); ``proj`` (activation type) one logit per head at b_off; ``dt`` [T, heads * dim] (activation
     type) the decay's argument, ``dt_bias`` float32 [heads * dim], ``a_log`` float32 [heads].  Returns float32 [T, P],
     P = 2 G d + H d + H + G:  q / sqrt(|q|^2 + unit_eps) * d^-1/2  |  k / sqrt(|k|^2 + unit_eps)  |
     exp(-exp(a_log) softplus(dt + dt_bias))  |  sigmoid(logit)  |  k . q.  ``per_head``: one decay a head instead of one a row
-    of its memory (``dt`` [T, heads], ``dt_bias`` [heads]; P = 2 G d + H + H + G)."""
+    of its memory (``dt`` [T, heads], ``dt_bias`` [heads]), and P = 2 G d + 4 H + 8 G:  q | k | per head: decay, beta, two unused |
+    per query/key head: q_t . k_(t-j) for j = 0 .. 3, k_t . k_(t-j) for j = 1 .. 3 with the rows before this one, one unused; all but
+    the first only from DELTA_BLOCK_MIN_TOKENS on (``max_q_len``, the longest segment).  What is unused is not written."""
     _cuda(xc, proj, dt, dt_bias, a_log)
     T = xc.shape[0]
     _f32_rows(xc, "delta_prepare: xc")
@@ -1598,26 +1603,29 @@ def delta_prepare(xc: torch.Tensor, q_off: int, k_off: int, proj: torch.Tensor, 
         raise KernelError("delta_prepare: a row is narrower than its heads")
     if a_log.dtype != torch.float32 or a_log.shape != (H,) or (dt_bias is not None and (dt_bias.dtype != torch.float32 or dt_bias.shape != (NA,))):
         raise KernelError("delta_prepare: a_log float32 [heads], dt_bias float32, one per decay")
-    prep = torch.empty((T, 2 * G * d + NA + H + G), dtype=torch.float32, device=xc.device)
+    prep = torch.empty((T, 2 * G * d + (4 * H + 8 * G if per_head else H * d + H + G)), dtype=torch.float32, device=xc.device)
     _check(library().pico_delta_prepare(_ptr(xc), xc.stride(0), q_off, k_off, _ptr(proj), proj.stride(0), b_off, _ptr(dt),
                                         dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(prep), T, H, G, d, float(d) ** -0.5,
-                                        float(unit_eps), 1 if per_head else 0, _dtype_code(proj), _stream()), "delta_prepare")
+                                        float(unit_eps), 1 if per_head else 0, 1 if max_q_len >= DELTA_BLOCK_MIN_TOKENS else 0,
+                                        _dtype_code(proj), _stream()), "delta_prepare")
     _count()
     return prep
 
 
 def gated_delta_rule(prep: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seg_slots: torch.Tensor, cu_q: torch.Tensor,
-                     positions: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, per_head: bool = False) -> torch.Tensor:
+                     positions: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, per_head: bool = False,
+                     max_q_len: int = 1) -> torch.Tensor:
     """Per head h, token by token in the order of each segment, from and into ``state`` float32 [slots, heads, vdim, dim] (S
     transposed; row ``seg_slots[s]``):  S <- diag(a) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.  ``prep``: the rows
-    :func:`delta_prepare` made with the same ``per_head`` (head h reads query and key head h // (heads / kv_heads)); ``v`` float32 rows with head h's values
+    :func:`delta_prepare` made with the same ``per_head`` and ``max_q_len`` (with a decay
+    per head and segments of DELTA_BLOCK_MIN_TOKENS and more, four tokens share one pass over the memory; head h reads query and key head h // (heads / kv_heads)); ``v`` float32 rows with head h's values
     at h * vdim (a column slice is fine).  A segment whose first position is negative is padding.  Returns o float32
     [T, heads * vdim]."""
     _cuda(prep, v, state, seg_slots, cu_q, positions)
     _f32_rows(v, "gated_delta_rule: v")
     T, S = prep.shape[0], seg_slots.shape[0]
     H, G, d = heads, kv_heads, dim
-    if prep.dtype != torch.float32 or not prep.is_contiguous() or prep.shape[1] != 2 * G * d + (H if per_head else H * d) + H + G or v.shape[0] != T \
+    if prep.dtype != torch.float32 or not prep.is_contiguous() or prep.shape[1] != 2 * G * d + (4 * H + 8 * G if per_head else H * d + H + G) or v.shape[0] != T \
             or v.shape[1] < H * vdim:
         raise KernelError("gated_delta_rule: prep must be what delta_prepare returns and v hold every head's values")
     if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (H, vdim, d):
@@ -1631,7 +1639,8 @@ def gated_delta_rule(prep: torch.Tensor, v: torch.Tensor, state: torch.Tensor, s
         raise KernelError("gated_delta_rule: cu_q must have one more entry than seg_slots, positions one per token")
     out = torch.empty((T, H * vdim), dtype=torch.float32, device=prep.device)
     _check(library().pico_gated_delta_rule(_ptr(prep), _ptr(v), v.stride(0), _ptr(state), _ptr(seg_slots), _ptr(cu_q),
-                                           _ptr(positions), _ptr(out), out.stride(0), S, H, G, d, vdim, 1 if per_head else 0, _stream()),
+                                           _ptr(positions), _ptr(out), out.stride(0), S, H, G, d, vdim, 1 if per_head else 0,
+                                           1 if max_q_len >= DELTA_BLOCK_MIN_TOKENS else 0, _stream()),
            f"gated_delta_rule (dim {d})")
     _count()
     return out

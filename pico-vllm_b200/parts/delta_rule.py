@@ -123,9 +123,10 @@ class GatedDeltaRule(Part):
         if self.head_decay:
             g0 = self.channels
             b0, a0 = g0 + H * dv, g0 + H * dv + H
-            prep = ops.delta_prepare(xc, 0, G * d, proj, b0, proj[:, a0:a0 + H], self.dt_bias, self.a_log, H, G, d, per_head=True)
+            prep = ops.delta_prepare(xc, 0, G * d, proj, b0, proj[:, a0:a0 + H], self.dt_bias, self.a_log, H, G, d, per_head=True,
+                                     max_q_len=batch.max_prefill_q)
             o = ops.gated_delta_rule(prep, xc[:, 2 * G * d:], memory.state, batch.seg_slots, batch.cu_q, batch.positions,
-                                     H, G, d, dv, per_head=True)
+                                     H, G, d, dv, per_head=True, max_q_len=batch.max_prefill_q)
             y = ops.group_rms_norm(o, H, dv, dv, self.out_norm, self.eps, h.dtype, post_gate=proj[:, g0:g0 + H * dv],
                                    post_act=self.gate_act)
             return _linear(y, self.o_weight)

@@ -620,7 +620,7 @@ NAMES = ["rotate_tail", "head_norm_store", "hyper_expand", "hyper_step", "scale_
          "gelu_gate_rows", "capped_glu", "tanh_norm", "map_rope_store", "map_difference", "bias_glu", "linear_bias", "skinny_gate_up_gelu"]
 
 
-def delta_prepare(xc, q_off, k_off, proj, b_off, dt, dt_bias, a_log, heads, kv_heads, dim, unit_eps=1e-6, per_head=False):
+def delta_prepare(xc, q_off, k_off, proj, b_off, dt, dt_bias, a_log, heads, kv_heads, dim, unit_eps=1e-6, per_head=False, max_q_len=1):
     T, H, G, d = xc.shape[0], heads, kv_heads, dim
     q = xc[:, q_off:q_off + G * d].reshape(T, G, d)
     k = xc[:, k_off:k_off + G * d].reshape(T, G, d)
@@ -629,15 +629,28 @@ def delta_prepare(xc, q_off, k_off, proj, b_off, dt, dt_bias, a_log, heads, kv_h
     z = dt.float() + (dt_bias if dt_bias is not None else 0.0)
     keep = torch.exp(-torch.exp(a_log).repeat_interleave(1 if per_head else d) * torch.nn.functional.softplus(z, threshold=20.0))
     beta = torch.sigmoid(proj[:, b_off:b_off + H].float())
+    if per_head:           # zeros where the kernel writes nothing
+        back = lambda j: torch.cat([torch.zeros(min(j, T), G, d), k[:max(T - j, 0)]])
+        dots = torch.zeros(T, G, 8)
+        for j in range(4 if max_q_len >= 4 else 1):
+            dots[:, :, j] = (q * back(j)).sum(-1)
+            if j:
+                dots[:, :, 3 + j] = (k * back(j)).sum(-1)
+        pair = torch.zeros(T, H, 4)
+        pair[:, :, 0], pair[:, :, 1] = keep, beta
+        return torch.cat([q.reshape(T, -1), k.reshape(T, -1), pair.reshape(T, -1), dots.reshape(T, -1)], 1).contiguous()
     return torch.cat([q.reshape(T, -1), k.reshape(T, -1), keep, beta, (q * k).sum(-1)], 1).contiguous()
 
 
-def gated_delta_rule(prep, v, state, seg_slots, cu_q, positions, heads, kv_heads, dim, vdim, per_head=False):
+def gated_delta_rule(prep, v, state, seg_slots, cu_q, positions, heads, kv_heads, dim, vdim, per_head=False, max_q_len=1):
     T, H, G, d = prep.shape[0], heads, kv_heads, dim
     q, k = prep[:, :G * d].reshape(T, G, d), prep[:, G * d:2 * G * d].reshape(T, G, d)
-    NA = H if per_head else H * d
-    keep = prep[:, 2 * G * d:2 * G * d + NA].reshape(T, H, -1)
-    beta = prep[:, 2 * G * d + NA:2 * G * d + NA + H]
+    if per_head:
+        keep, beta = prep[:, 2 * G * d:2 * G * d + 4 * H].reshape(T, H, 4)[:, :, :2].split(1, 2)
+        beta = beta[:, :, 0]
+    else:
+        keep = prep[:, 2 * G * d:2 * G * d + H * d].reshape(T, H, d)
+        beta = prep[:, 2 * G * d + H * d:2 * G * d + H * d + H]
     out = torch.zeros(T, H * vdim)
     for s in range(seg_slots.shape[0]):
         a0, a1 = int(cu_q[s]), int(cu_q[s + 1])

@@ -266,9 +266,15 @@ def _segments(lens, pad_at=None):
 
 
 @pytest.mark.parametrize("H,G,d,dv", [(4, 2, 16, 24), (2, 2, 40, 8), (3, 1, 64, 64), (2, 1, 200, 130), (1, 1, 128, 16), (6, 3, 10, 20)])
-@pytest.mark.parametrize("lens,pad_at", [([1, 70, 5, 2], 2), ([1, 1, 1], None), ([33], None)])
+@pytest.mark.parametrize("lens,pad_at", [([1, 70, 5, 2], 2), ([1, 1, 1], None), ([33], None), ([3, 2, 3], None), ([4, 1, 15, 16, 17], None)])
 def test_delta_rule_kernels_with_a_decay_per_head(H, G, d, dv, lens, pad_at):
+    """Both forms: a pass over the memory for every token, and for every four (steps that hold a segment of four or more)."""
     from pico_vllm_b200 import ops
+    for longest in (1, max(lens)):
+        _delta_rule_case(ops, H, G, d, dv, lens, pad_at, longest)
+
+
+def _delta_rule_case(ops, H, G, d, dv, lens, pad_at, longest):
     g = torch.Generator().manual_seed(d + dv + len(lens))
     cu, pos, seg, slots = _segments(lens, pad_at)
     T, S = int(cu[-1]), len(lens)
@@ -277,17 +283,22 @@ def test_delta_rule_kernels_with_a_decay_per_head(H, G, d, dv, lens, pad_at):
     dt_bias, a_log = torch.randn(H, generator=g), torch.randn(H, generator=g) - 1.0
     for dtype in (torch.float32, torch.bfloat16):
         p = proj.to(dtype)
-        want = fake_ops.delta_prepare(xc, 2, 2 + G * d, p, 3, p[:, 3 + H:3 + 2 * H], dt_bias, a_log, H, G, d, per_head=True)
+        want = fake_ops.delta_prepare(xc, 2, 2 + G * d, p, 3, p[:, 3 + H:3 + 2 * H], dt_bias, a_log, H, G, d, per_head=True, max_q_len=longest)
         pg = p.to(DEV)
-        got = ops.delta_prepare(xc.to(DEV), 2, 2 + G * d, pg, 3, pg[:, 3 + H:3 + 2 * H], dt_bias.to(DEV), a_log.to(DEV), H, G, d, per_head=True)
+        got = ops.delta_prepare(xc.to(DEV), 2, 2 + G * d, pg, 3, pg[:, 3 + H:3 + 2 * H], dt_bias.to(DEV), a_log.to(DEV), H, G, d, per_head=True,
+                                max_q_len=longest).cpu()
+        pair, dots = got[:, 2 * G * d:2 * G * d + 4 * H].view(T, H, 4), got[:, 2 * G * d + 4 * H:].view(T, G, 8)
+        pair[:, :, 2:] = 0                             # numbers nobody reads
+        dots[:, :, 7 if longest >= ops.DELTA_BLOCK_MIN_TOKENS else 1:] = 0
         _close(got, want, 2e-6, "delta_prepare")
     prep = want
     state = torch.randn(S + 1, H, dv, d, generator=g) * 0.3
     v = xc[:, 2 + 2 * G * d:]
     st_want = state.clone()
-    o_want = fake_ops.gated_delta_rule(prep, v, st_want, slots, cu, pos, H, G, d, dv, per_head=True)
+    o_want = fake_ops.gated_delta_rule(prep, v, st_want, slots, cu, pos, H, G, d, dv, per_head=True, max_q_len=longest)
     st_got = state.to(DEV)
-    o_got = ops.gated_delta_rule(prep.to(DEV), v.to(DEV), st_got, slots.to(DEV), cu.to(DEV), pos.to(DEV), H, G, d, dv, per_head=True)
+    o_got = ops.gated_delta_rule(prep.to(DEV), v.to(DEV), st_got, slots.to(DEV), cu.to(DEV), pos.to(DEV), H, G, d, dv, per_head=True,
+                                 max_q_len=longest)
     live = pos >= 0
     _close(o_got.cpu()[live], o_want[live], 2e-5, "delta rule outputs")
     _close(st_got, st_want, 2e-5, "delta rule states")
