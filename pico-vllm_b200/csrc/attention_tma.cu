@@ -65,6 +65,8 @@ __device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* map, i
         : "memory");
 }
 // thread-block cluster: barrier over all threads of all blocks, and loads from another block's shared memory
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.relaxed.aligned;\n" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory"); }
 __device__ __forceinline__ void cluster_sync_all() {
     asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
     asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
@@ -114,6 +116,10 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     // kv_same: keys and values are one tensor (a cached latent that serves as both): only the key tile is copied and
     // the p.v product reads it too - the two maps give tiles of the same layout
     pdl_launch_dependents();
+    // Another block's shared memory may be written only once that block runs: every thread reports here that its block does and
+    // waits, before the partial results are pushed, until all blocks of the cluster have.  (The parts of a key range differ in
+    // length; a short or empty one would otherwise push into a block that has not started, which is a fault.)
+    if (cluster_reduce) cluster_arrive();
     extern __shared__ unsigned char smem_dyn[];
     constexpr int TILE_BYTES = MMA_BN * HD * 2;                  // one K or V tile
     constexpr int QLD = HD + 8;
@@ -201,7 +207,11 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
                             full + s);
             }
         }
-        if (cluster_reduce) cluster_sync_all();     // every thread of the cluster takes part in its barrier
+        if (cluster_reduce) {                       // every thread of the cluster takes part in its barriers
+            __syncwarp();
+            cluster_wait();
+            cluster_sync_all();
+        }
         return;
     }
     // -------------------------------------------------------------------- consumers (warps 0..CW-1)
@@ -388,6 +398,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
             }
         }
     consumer_sync<CW * 32>();
+    if (cluster_reduce) cluster_wait();             // all blocks of the cluster run: their shared memory may be written
     const float LN2 = 0.6931471805599453f;
     // With a cluster, block sp adds output elements [sp * share, (sp + 1) * share) of the g * HD over all
     // blocks: every block PUSHES what it has of another block's share (and its maxima and sums) into
